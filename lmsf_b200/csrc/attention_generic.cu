@@ -40,6 +40,7 @@ struct GenericAttnArgs {
   int keep_first;                              // > 0 (with a window): the first keep_first keys of the request stay visible behind the window
   int sigmoid;                                 // 1: a key's weight is sigmoid(score), not normalised over the keys (no softmax)
   const float* head_bias;                      // [n_q_heads] or null: a number per query head added to every scaled score
+  const float* dist; int dist_n;               // [n_q_heads][dist_n] or null: the entry of (query position - key position), the last for larger ones, is added
 };
 
 template <typename T>
@@ -94,6 +95,7 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
         if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
         if (a.slopes) s = fmaf(a.slopes[head], (float)(key - pos), s);
         if (a.log_r1) s -= a.log_r1[head] * logf(1.0f + a.log_r2[head] * (float)(pos - key));
+        if (a.dist) s += a.dist[(size_t)head * a.dist_n + min(pos - key, a.dist_n - 1)];
         s += hb;
       }
     }
@@ -179,14 +181,16 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
 // keep_first > 0 (with a window): the request's first keep_first keys stay visible when the window has passed them, at their
 // true positions.  sigmoid = 1: a visible key's weight is sigmoid(score) and the weights are not normalised (no softmax; sinks
 // have no meaning then).  head_bias ([n_q_heads] float32 or null): added to every scaled score of its head.
-LMSF_API int lmsf_attention_generic_weights(const void* q, long long q_stride, void* out, long long out_stride,
-                                            const void* cache, long long page_stride, const int* block_table, int max_blocks,
-                                            int block_size, const int* token_seq, const int* positions, float scale,
-                                            float softcap, const float* slopes, int window, int n_tokens, int n_q_heads,
-                                            int n_kv_heads, int head_dim, int dtype, int shared_kv, const void* gate,
-                                            long long gate_stride, int chunk, const float* log_r1, const float* log_r2,
-                                            const float* sinks, int keep_first, int sigmoid, const float* head_bias,
-                                            void* stream) {
+// dist ([n_q_heads][dist_n] float32 or null): a table of what is added to the scaled score by (query position - key position);
+// its last entry serves every larger distance.
+LMSF_API int lmsf_attention_generic_dist(const void* q, long long q_stride, void* out, long long out_stride,
+                                         const void* cache, long long page_stride, const int* block_table, int max_blocks,
+                                         int block_size, const int* token_seq, const int* positions, float scale,
+                                         float softcap, const float* slopes, int window, int n_tokens, int n_q_heads,
+                                         int n_kv_heads, int head_dim, int dtype, int shared_kv, const void* gate,
+                                         long long gate_stride, int chunk, const float* log_r1, const float* log_r2,
+                                         const float* sinks, int keep_first, int sigmoid, const float* head_bias,
+                                         const float* dist, int dist_n, void* stream) {
   using namespace lmsf;
   if (n_tokens <= 0) return 0;
   if (head_dim <= 0 || head_dim > kMaxHeadDim || head_dim % 16)
@@ -200,13 +204,28 @@ LMSF_API int lmsf_attention_generic_weights(const void* q, long long q_stride, v
   GenericAttnArgs a{q, q_stride, out, out_stride, cache, page_stride, block_table, max_blocks, block_size,
                     token_seq, positions, scale, window, n_q_heads, n_kv_heads, head_dim, softcap > 0.f ? softcap : 0.f, slopes,
                     shared_kv ? 1 : 0, gate, gate_stride, chunk > 0 ? chunk : 0, log_r1, log_r2, sinks,
-                    (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias};
+                    (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
+  if (dist && dist_n <= 0) LMSF_REFUSE("attention: a table of %d distances", dist_n);
   if (sigmoid && sinks) LMSF_REFUSE("attention: sinks belong to a softmax, not to sigmoid weights");
   dim3 grid(n_tokens, n_q_heads);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == LMSF_F32) attention_generic_kernel<float><<<grid, kWarps * 32, 0, s>>>(a);
   else attention_generic_kernel<bf16><<<grid, kWarps * 32, 0, s>>>(a);
   return LMSF_LAUNCH_STATUS();
+}
+
+LMSF_API int lmsf_attention_generic_weights(const void* q, long long q_stride, void* out, long long out_stride,
+                                            const void* cache, long long page_stride, const int* block_table, int max_blocks,
+                                            int block_size, const int* token_seq, const int* positions, float scale,
+                                            float softcap, const float* slopes, int window, int n_tokens, int n_q_heads,
+                                            int n_kv_heads, int head_dim, int dtype, int shared_kv, const void* gate,
+                                            long long gate_stride, int chunk, const float* log_r1, const float* log_r2,
+                                            const float* sinks, int keep_first, int sigmoid, const float* head_bias,
+                                            void* stream) {
+  return lmsf_attention_generic_dist(q, q_stride, out, out_stride, cache, page_stride, block_table, max_blocks, block_size,
+                                     token_seq, positions, scale, softcap, slopes, window, n_tokens, n_q_heads, n_kv_heads,
+                                     head_dim, dtype, shared_kv, gate, gate_stride, chunk, log_r1, log_r2, sinks, keep_first,
+                                     sigmoid, head_bias, nullptr, 0, stream);
 }
 
 LMSF_API int lmsf_attention_generic_masked(const void* q, long long q_stride, void* out, long long out_stride,

@@ -132,6 +132,12 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
     for (int h = 0; h < 2; ++h)
       if (g4 + h * 8 < n_heads) { r1[h] = a.x.r1[head0 + g4 + h * 8]; r2[h] = a.x.r2[head0 + g4 + h * 8]; }
   }
+  const float* dist_row[2] = {a.x.dist, a.x.dist};             // the heads' rows of a table of distances, if there is one
+  if (a.x.dist) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      if (g4 + h * 8 < n_heads) dist_row[h] = a.x.dist + (size_t)(head0 + g4 + h * 8) * a.x.dist_n;
+  }
   float hb2[2] = {0.f, 0.f};                                   // the heads' biases on the scores, in base-2 units
   if (a.x.head_bias) {
 #pragma unroll
@@ -230,6 +236,7 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
         const bool ok = (key >= lo || key < keep) && key < ctx;
         float v = ok ? fmaf(s[j][e], sl2, hb2[e >> 1]) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2(r1[e >> 1], r2[e >> 1], ctx - 1 - key);
+        if (dist_row[0] && ok) v += table_bias2(dist_row[e >> 1], a.x.dist_n, ctx - 1 - key);
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -617,7 +624,8 @@ LMSF_API int lmsf_attention_decode_width(const void* q, long long q_stride, void
                                          int n_seqs_total, const int* cu_q, const int* ctx_len, float scale, int window,
                                          int n_q_heads, int head_dim, int n_splits, int block_warps, void* scratch,
                                          int kv_planes, int chunk, const float* r1, const float* r2, const float* sinks,
-                                         int keep_first, int sigmoid, const float* head_bias, void* stream) {
+                                         int keep_first, int sigmoid, const float* head_bias, const float* dist, int dist_n,
+                                         void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (n_served <= 0) return 0;
@@ -647,7 +655,8 @@ LMSF_API int lmsf_attention_decode_width(const void* q, long long q_stride, void
   a.scale = scale; a.window = window; a.n_q_heads = n_q_heads; a.group = group; a.n_splits = n_splits;
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_decode: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_decode: sinks belong to a softmax, not to sigmoid weights");
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias};
+  if (dist && dist_n <= 0) LMSF_REFUSE("attention_decode: a table of %d distances", dist_n);
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   a.rows = decode_rows(group);
   if (block_warps != 0 && block_warps != 2 && block_warps != 4)
     LMSF_REFUSE("attention_decode: blocks have 2 or 4 warps, not %d", block_warps);
@@ -728,7 +737,7 @@ LMSF_API int lmsf_attention_decode_items(const void* q, long long q_stride, void
                                          int n_seqs_total, const int* cu_q, const int* ctx_len, float scale, int window,
                                          int n_q_heads, int head_dim, int block_warps, void* scratch, int kv_planes,
                                          int chunk, const float* r1, const float* r2, const float* sinks, int keep_first,
-                                         int sigmoid, const float* head_bias, void* stream) {
+                                         int sigmoid, const float* head_bias, const float* dist, int dist_n, void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (capacity <= 0) return 0;
@@ -755,7 +764,8 @@ LMSF_API int lmsf_attention_decode_items(const void* q, long long q_stride, void
   a.scale = scale; a.window = window; a.n_q_heads = n_q_heads; a.group = group; a.n_splits = 1;
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_decode: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_decode: sinks belong to a softmax, not to sigmoid weights");
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias};
+  if (dist && dist_n <= 0) LMSF_REFUSE("attention_decode: a table of %d distances", dist_n);
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   a.rows = decode_rows(group);
   a.items = (const int4*)items;
   a.cluster = 0;
@@ -771,7 +781,7 @@ LMSF_API int lmsf_attention_decode(const void* q, long long q_stride, void* out,
                                    int n_q_heads, int head_dim, int n_splits, void* scratch, void* stream) {
   return lmsf_attention_decode_width(q, q_stride, out, out_stride, cache, page_stride, block_size, n_kv_heads, block_table,
                                      max_blocks, seq_ids, n_served, n_seqs_total, cu_q, ctx_len, scale, window, n_q_heads,
-                                     head_dim, n_splits, 0, scratch, 2, 0, nullptr, nullptr, nullptr, 0, 0, nullptr, stream);
+                                     head_dim, n_splits, 0, scratch, 2, 0, nullptr, nullptr, nullptr, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 // ------------------------------------------------------------------------------------------------

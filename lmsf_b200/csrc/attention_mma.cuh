@@ -69,6 +69,8 @@ struct ScoreExtras {
   int keep_first;       // > 0 (with a window): the request's first keep_first keys stay visible behind the window
   int sigmoid;          // 1: a visible key's weight is sigmoid(score), not normalised over the keys (no softmax, no sinks)
   const float* head_bias;   // [n_q_heads]: a number per query head added to every scaled score
+  const float* dist;        // [n_q_heads][dist_n]: the entry of the distance p - key (the last entry for every distance from
+  int dist_n;               // dist_n - 1 on) is added to the scaled score
 };
 // The key tiles that a block walks when the window's keys [lo, hi) are joined by the kept first keys [0, keep): tiles
 // 0 .. n_first - 1 and then tile_lo .. tile_hi - 1 (n_first = 0 when the window's first tile reaches the kept keys anyway).
@@ -90,6 +92,10 @@ __device__ __forceinline__ float sigmoid2(float v) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-v));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
   return r;
+}
+// what a table of distances adds to a score, in base-2 units; `row` is the head's row of the table
+__device__ __forceinline__ float table_bias2(const float* __restrict__ row, int n, int distance) {
+  return row[min(max(distance, 0), n - 1)] * 1.4426950408889634f;
 }
 // the first key that a query at position p sees
 __device__ __forceinline__ int first_seen(int p, int window, int chunk) {

@@ -49,6 +49,7 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   const int keep = a.x.keep_first;                               // keys below it are seen behind the window too
   const bool sig = a.x.sigmoid != 0;
   const float hb2 = a.x.head_bias ? a.x.head_bias[head] * kLog2e : 0.f;
+  const float* dist_row = a.x.dist ? a.x.dist + (size_t)head * a.x.dist_n : nullptr;
   const int warp_last_pos = start + q0 + min(warp * 16 + 15, rows_valid - 1);
   const int warp_first_pos = start + q0 + min(warp * 16, rows_valid - 1);
   const int warp_lo = first_seen(warp_first_pos, a.window, a.x.chunk);
@@ -118,6 +119,7 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
         const bool ok = key <= pos[h] && (key >= row_lo[h] || key < keep);
         float v = ok ? fmaf(s[j][e], sl2, hb2) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2f(r1, r2, dist0[h] - (float)(j * 8 + (e & 1)));
+        if (dist_row && ok) v += table_bias2(dist_row, a.x.dist_n, pos[h] - key);
         s[j][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -192,7 +194,7 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
                                     int n_tiles, const int* cu_q, const int* ctx_len, float scale, int window,
                                     int n_q_heads, int head_dim, int kv_planes, int chunk, const float* r1,
                                     const float* r2, const float* sinks, int keep_first, int sigmoid,
-                                    const float* head_bias, void* stream) {
+                                    const float* head_bias, const float* dist, int dist_n, void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (n_tiles <= 0) return 0;
@@ -210,7 +212,8 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
   a.group = n_q_heads / n_kv_heads;
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_prefill: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_prefill: sinks belong to a softmax, not to sigmoid weights");
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias};
+  if (dist && dist_n <= 0) LMSF_REFUSE("attention_prefill: a table of %d distances", dist_n);
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   const int smem = kStages * St::kBytes;
   static bool configured = false;
   if (!configured) {

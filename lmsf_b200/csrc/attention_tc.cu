@@ -608,19 +608,22 @@ __global__ void __launch_bounds__(kThreadsTotal, 1) prefill_tc_kernel(const Args
 #pragma unroll
         for (int c0 = 0; c0 < BN; c0 += 32) tmem_ld32_issue(t_s + c0, sc + c0);
         tmem_wait_ld();
-        if (a.x.r1 != nullptr) {
+        if (a.x.r1 != nullptr || a.x.dist != nullptr) {
           // The bias is taken off the raw scores, in their own units (the scale is folded in below, with the maximum).
           // It depends on the distance alone, and the 32 rows of a warp meet the tile's 128 keys at 159 distances: the
           // warp computes those once (five logarithms a thread instead of 128) into its own table, and every score
           // costs a shared-memory load and a subtraction.  Entry t is the distance (first row of the warp) - (last key
           // of the tile) + t; row l and key i meet at t = l + BN - 1 - i, so the lanes of a warp read consecutive words.
-          // The constants are read here, tile by tile, so that they hold no register where there is no bias.
-          const float r1s = a.x.r1[note->head] / sl2, r2 = a.x.r2[note->head];
+          // The constants are read here, tile by tile, so that they hold no register where there is no bias.  A table of
+          // distances is spread out in the same way (negated, in the raw scores' units).
           float* tbl = bias_tbl[warp];
           const int d_first = q_pos0 + (row & ~31) - key0 - (BN - 1);
           __syncwarp();                                                // the tile before has been read
 #pragma unroll
-          for (int t = lane; t < kBiasEntries; t += 32) tbl[t] = log_distance_bias2(r1s, r2, d_first + t);
+          for (int t = lane; t < kBiasEntries; t += 32) {
+            if (a.x.dist != nullptr) tbl[t] = -a.x.dist[(size_t)note->head * a.x.dist_n + min(max(d_first + t, 0), a.x.dist_n - 1)] / a.scale;
+            else tbl[t] = log_distance_bias2(a.x.r1[note->head] / sl2, a.x.r2[note->head], d_first + t);
+          }
           __syncwarp();
           const float* mine = tbl + lane + (BN - 1);
 #pragma unroll
@@ -802,7 +805,7 @@ LMSF_API int lmsf_attention_prefill_tc(const void* q, long long q_stride, long l
                                        int n_tiles, const int* cu_q, const int* ctx_len, float scale, int window,
                                        int n_q_heads, int head_dim, int* error_flag, int kv_planes, int chunk,
                                        const float* r1, const float* r2, const float* sinks, int keep_first, int sigmoid,
-                                       const float* head_bias, void* stream) {
+                                       const float* head_bias, const float* dist, int dist_n, void* stream) {
   using namespace lmsf;
   using namespace lmsf::tc;
   if (n_tiles <= 0) return 0;
@@ -826,7 +829,9 @@ LMSF_API int lmsf_attention_prefill_tc(const void* q, long long q_stride, long l
     LMSF_REFUSE("attention_prefill_tc: the distance bias takes both constants and a positive scale; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_prefill_tc: sinks belong to a softmax, not to sigmoid weights");
   if (!sigmoid && head_bias) LMSF_REFUSE("attention_prefill_tc: a bias per head is taken with sigmoid weights only");
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias};
+  if (dist && (dist_n <= 0 || !(scale > 0.f) || r1))
+    LMSF_REFUSE("attention_prefill_tc: a table of distances has entries, a positive scale and no other distance bias beside it");
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   // pages of 8 keys and more come by tensor-map copies (a box of rows_box keys starts on a 1024-byte
   // boundary of the swizzled tile); smaller pages by cp.async
   a.rows_box = block_size < BN ? block_size : BN;

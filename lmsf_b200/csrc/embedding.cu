@@ -40,6 +40,29 @@ __global__ void embedding_scaled_kernel(T* __restrict__ out, const T* __restrict
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? from_f32<T>(to_f32(src[i]) * scale) : from_f32<T>(0.f);
 }
 
+// The same as the start of a float32 residual stream: the product is not rounded, whatever the table's type.
+template <typename T, int V>
+__global__ void embedding_stream_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
+                                        int hidden, int vocab, float scale, int* __restrict__ error_flag) {
+  const int t = blockIdx.x;
+  const int id = ids[t];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0 && error_flag) atomicExch(error_flag, 1);
+  const T* src = table + (size_t)(ok ? id : 0) * hidden;
+  float* dst = out + (size_t)t * hidden;
+  for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      float x[4];
+      ld4(src + i, x);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) x[k] = ok ? x[k] * scale : 0.f;
+      st4(dst + i, x);
+    } else {
+      dst[i] = ok ? to_f32(src[i]) * scale : 0.f;
+    }
+  }
+}
+
 // out[t, :] = table[id_t, :] * scale + pairs[row_t, :] in float32, where row_t = (id_{t-1} * mul_prev + id_t * mul_cur) mod buckets
 // is chosen by the token and the token before it in the same request, and row `buckets` (the table's last) belongs to a
 // request's first token.  The token before a portion's first token is the request's state: last[slot], one int32 per state
@@ -166,5 +189,22 @@ LMSF_API int lmsf_embedding_pairs(float* out, const void* table, const void* pai
   else if (dtype == LMSF_BF16) { if (vec) LMSF_EP(bf16, true); else LMSF_EP(bf16, false); }
   else LMSF_REFUSE("embedding: unknown dtype code %d", dtype);
 #undef LMSF_EP
+  return LMSF_LAUNCH_STATUS();
+}
+
+// out: float32 [n, hidden] = table[ids] * scale, the start of a float32 residual stream; table: [vocab, hidden] of `dtype`.
+LMSF_API int lmsf_embedding_stream(float* out, const void* table, const int* ids, int n, int hidden, int vocab, float scale,
+                                   int dtype, int* error_flag, void* stream) {
+  using namespace lmsf;
+  if (n <= 0) return 0;
+  if (hidden <= 0 || vocab <= 0) LMSF_REFUSE("embedding_stream: hidden=%d vocab=%d", hidden, vocab);
+  if (dtype != LMSF_F32 && dtype != LMSF_BF16) LMSF_REFUSE("embedding_stream: unknown dtype code %d", dtype);
+  cudaStream_t s = (cudaStream_t)stream;
+  const int threads = hidden >= 1024 ? 256 : 64;
+  const bool wide = hidden % 4 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)table % (dtype == LMSF_F32 ? 16 : 8) == 0;
+#define LMSF_GO(T, V) embedding_stream_kernel<T, V><<<n, threads, 0, s>>>(out, (const T*)table, ids, hidden, vocab, scale, error_flag)
+  if (dtype == LMSF_F32) { if (wide) LMSF_GO(float, 4); else LMSF_GO(float, 1); }
+  else { if (wide) LMSF_GO(bf16, 4); else LMSF_GO(bf16, 1); }
+#undef LMSF_GO
   return LMSF_LAUNCH_STATUS();
 }

@@ -63,6 +63,9 @@ struct Args {
   // residual form: res[m, n] += bfloat16(sum); out[m, n] = bfloat16(res[m, n] * norm_w[n]);
   // out_sumsq[m * out_ld + block] = sum of res[m, n]^2 over the block's n
   float* res; long long ldres; const void* norm_w; int norm_w_f32; float* out_sumsq; long long out_ld;
+  const bf16* bias;   // [N] or null: added to the sums before anything else is done with them (plain and ROPE forms)
+  int plain_act;      // plain form: 0 none, 1 the square of max(sum, 0)
+  int planes;         // ROPE: 2 (k and v rows) or 1 (k rows only: a cache whose keys are its values)
 };
 
 __device__ __forceinline__ float act_apply(float g, int act) {
@@ -128,7 +131,7 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
   auto issue_w = [&](int c) {
     const uint32_t st = ring + (c % STAGES) * kStage;
     const int k0 = (c_begin + c * c_stride) * kChunkK;
-    if (ROPE) issue_rows<16>(st, a.w + (size_t)f0 * a.ldw, a.ldw, 16, k0, a.K, lane, hi_off);
+    if (ROPE) issue_rows<16>(st, a.w + (size_t)f0 * a.ldw, a.ldw, pair8 ? 16 : min(16, a.N - f0), k0, a.K, lane, hi_off);
     else if (PAIR) issue_rows<16>(st, a.w + (size_t)n0 * a.ldw, a.ldw, min(8, rows_total - n0), k0, a.K, lane, a.up_offset - 8, true);
     else issue_rows<16>(st, a.w + (size_t)n0 * a.ldw, a.ldw, rows_total - n0, k0, a.K, lane);
     if (GROUPS == 2)
@@ -194,7 +197,7 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
       const int m = (threadIdx.x + t * kWarps * 32) / 16;
       e_pos[t] = m < a.M ? a.positions[m] : 0;
       e_page[t] = -1;
-      if (m < a.M && f0 >= a.n_q_heads * a.head_dim) {            // a block of k or v features
+      if (m < a.M && f0 >= a.n_q_heads * a.head_dim && f0 < (a.n_q_heads + a.planes * a.n_kv_heads) * a.head_dim) {   // a block of k or v features
         const int blk = e_pos[t] / a.block_size;
         e_page[t] = blk < a.max_blocks ? a.block_table[(size_t)a.token_seq[m] * a.max_blocks + blk] : -1;
       }
@@ -295,12 +298,17 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
       for (int w = 0; w < kWarps; ++w)
         sum += reinterpret_cast<const float*>(smem + w * (STAGES * kStage))[row * (8 * NT) + m];
       sum *= factor(m);
+      const int n = row < 8 ? f0 + row : f1 + row - 8;                  // feature among q, k, v (and the rows behind them)
+      if (a.bias && n < a.N) sum += __bfloat162float(a.bias[n]);
       const float val = __bfloat162float(__float2bfloat16_rn(sum));      // what the plain product would have stored
       const float other = __shfl_xor_sync(0xffffffffu, val, pair8 ? 8 : 1);
-      if (m >= a.M) continue;
-      const int n = row < 8 ? f0 + row : f1 + row - 8;                  // feature among q, k, v
+      if (m >= a.M || n >= a.N) continue;
       const int d = n % a.head_dim;
       const bool is_v = n >= q_size + kv_size;
+      if (n >= q_size + a.planes * kv_size) {                            // a row that only passes: its own column of out
+        reinterpret_cast<bf16*>(a.out)[(size_t)m * a.ldo + n] = __float2bfloat16_rn(val);
+        continue;
+      }
       float r = val;
       if (a.inv_freq && !is_v && d < a.rot_dim) {
         const bool first = a.is_neox ? d < a.rot_dim / 2 : (d & 1) == 0;
@@ -353,7 +361,11 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
           s += reinterpret_cast<const float*>(smem + w * (STAGES * kStage))[g * (16 * 8 * NT) + row * (8 * NT) + m];
         v[g] = s * f;
       }
-      const float r = GROUPS == 2 ? act_apply(v[0], a.act) * v[GROUPS - 1] : v[0];
+      float r = GROUPS == 2 ? act_apply(v[0], a.act) * v[GROUPS - 1] : v[0];
+      if (GROUPS == 1) {
+        if (a.bias && ok) r += __bfloat162float(a.bias[n0 + row]);
+        if (a.plain_act) { r = fmaxf(r, 0.f); r *= r; }
+      }
       if (GROUPS == 1 && a.res) {
         float nr = 0.f;
         if (ok) {
@@ -482,14 +494,18 @@ static int run_product(Args& a, int fuse_act, cudaStream_t s) {
 // x: [M, K] bfloat16 (M <= 16), w: [N, K] bfloat16, out: [M, N] bfloat16 or float32.  K % 8 == 0.
 // fuse_act < 0: plain product.  fuse_act = 0 (silu) or 1 (gelu_tanh): w is [2 * N_out, K] (gate rows first),
 // out is [M, N_out] = act(x gate^T) * (x up^T), N = 2 * N_out.
+// bias (bfloat16 [N], may be null) is added to the sums; plain_act = 1: the result is the square of max(sum, 0) (plain product).
 // in_sumsq (may be null): x is a prenormed input, a residual stream times a norm weight; the sums of token m are
 // multiplied by 1 / sqrt(sum of in_sumsq[m * in_ld + 0 .. in_parts) / in_width + in_eps) first.
 LMSF_API int lmsf_gemm_skinny(void* out, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
                               long long ldo, int fuse_act, int out_f32, const float* in_sumsq, int in_parts,
-                              long long in_ld, float in_eps, int in_width, void* stream) {
+                              long long in_ld, float in_eps, int in_width, const void* bias, int plain_act, void* stream) {
   using namespace lmsf;
   using namespace lmsf::skinny;
   Args a{};
+  if (fuse_act >= 0 && (bias || plain_act)) LMSF_REFUSE("gemm_skinny: a bias or an activation of the plain form beside a gated activation");
+  if (plain_act != 0 && plain_act != 1) LMSF_REFUSE("gemm_skinny: unknown activation code %d of the plain form", plain_act);
+  a.bias = (const bf16*)bias; a.plain_act = plain_act;
   a.x = (const bf16*)x; a.ldx = ldx; a.w = (const bf16*)w; a.ldw = ldw; a.out = out; a.ldo = ldo; a.M = M; a.N = N; a.K = K;
   a.out_f32 = out_f32;
   a.in_sumsq = in_sumsq; a.in_parts = in_parts; a.in_ld = in_ld; a.in_eps = in_eps; a.in_width = in_width;
@@ -519,13 +535,16 @@ LMSF_API int lmsf_gemm_skinny_residual(void* out, long long ldo, const void* x, 
 // epilogue.  w: [(n_q_heads + 2 n_kv_heads) * head_dim, K]; q_out: [M, n_q_heads * head_dim] bfloat16, rotated;
 // k (rotated) and v go to the pages of `cache` ([page][2][kv_head][slot][head_dim]) that block_table names for
 // positions[m] of request token_seq[m].  inv_freq: [rot_dim / 2] float32 or null (no rotation).  Results are those
-// of lmsf_gemm_skinny (bfloat16 out) followed by the rotary / cache-write kernel, bit for bit.  in_sumsq: as there.
+// of lmsf_gemm_skinny (bfloat16 out) followed by the rotary / cache-write kernel, bit for bit.  in_sumsq, bias: as there.
+// planes = 1: there are no v rows (the cache holds one vector per token and kv head, key and value at once).  n_extra: w has
+// so many rows behind q, k and v whose results go to their own columns of q_out, a row of which then spans all of w's rows.
 LMSF_API int lmsf_gemm_skinny_qkv_rope(void* q_out, long long ldq, const void* x, long long ldx, const void* w, long long ldw,
                                        int M, int K, const int* positions, const int* token_seq, const int* block_table,
                                        int max_blocks, int block_size, void* cache, long long page_stride,
                                        const float* inv_freq, int rot_dim, int is_neox, int n_q_heads, int n_kv_heads,
                                        int head_dim, int* error_flag, const float* in_sumsq, int in_parts,
-                                       long long in_ld, float in_eps, int in_width, void* stream) {
+                                       long long in_ld, float in_eps, int in_width, const void* bias, int planes, int n_extra,
+                                       void* stream) {
   using namespace lmsf;
   using namespace lmsf::skinny;
   if (M <= 0) return 0;
@@ -541,7 +560,10 @@ LMSF_API int lmsf_gemm_skinny_qkv_rope(void* q_out, long long ldq, const void* x
     LMSF_REFUSE("gemm_skinny_qkv_rope: bad q or cache geometry");
   Args a{};
   a.x = (const bf16*)x; a.ldx = ldx; a.w = (const bf16*)w; a.ldw = ldw; a.out = q_out; a.ldo = ldq;
-  a.M = M; a.N = (n_q_heads + 2 * n_kv_heads) * head_dim; a.K = K; a.act = -1;
+  if ((planes != 1 && planes != 2) || n_extra < 0 || (n_extra > 0 && ldq < (long long)(n_q_heads + planes * n_kv_heads) * head_dim + n_extra))
+    LMSF_REFUSE("gemm_skinny_qkv_rope: planes=%d, %d rows behind them (an output row must hold every row of w then)", planes, n_extra);
+  a.M = M; a.N = (n_q_heads + planes * n_kv_heads) * head_dim + n_extra; a.K = K; a.act = -1;
+  a.bias = (const bf16*)bias; a.planes = planes;
   a.positions = positions; a.token_seq = token_seq; a.block_table = block_table; a.max_blocks = max_blocks;
   a.block_size = block_size; a.cache = (bf16*)cache; a.page_stride = page_stride; a.inv_freq = inv_freq;
   a.rot_dim = inv_freq ? rot_dim : 0; a.is_neox = is_neox; a.n_q_heads = n_q_heads; a.n_kv_heads = n_kv_heads;

@@ -37,10 +37,25 @@ __global__ void __launch_bounds__(128) latent_norm_cache_write_kernel(const T* _
     dst[i] = i < rank ? from_f32<T>((to_f32(xr[i]) * inv) * w[i]) : from_f32<T>(0.f);
 }
 
+// How a rotated part of `n` values turns: value first(i) pairs with value second(i) for i < n / 2, the angle is position *
+// inv_freq[i] in float32, and both cos and sin are multiplied by `mult` (1 for a plain rotation).
+struct PartRotation {
+  const float* inv_freq; int n; int interleaved; float mult;
+  __device__ __forceinline__ int first(int i) const { return interleaved ? 2 * i : i; }
+  __device__ __forceinline__ int second(int i) const { return interleaved ? 2 * i + 1 : i + n / 2; }
+  __device__ __forceinline__ void angle(int pos, int i, float* cs, float* sn) const {
+    float c, s;
+    sincosf((float)pos * inv_freq[i], &s, &c);
+    *cs = c * mult;
+    *sn = s * mult;
+  }
+};
+
 // The same with a rotated key part behind the normed vector: a row of x holds rank values to norm and `rot_dim` values of
-// one key part that all heads share; of those the first `rot_n` are rotated by the token's position (value i pairs with
-// value i + rot_n / 2, angle = position * inv_freq[i], float32), the rest pass unchanged.  The page's row is
-// [normed vector | key part | zeros]: the attention reads it as one key (and value) of `padded` values.
+// one key part that all heads share; of those the first rot.n are rotated by the token's position, the rest pass unchanged.
+// The page's row is [normed vector | key part | zeros]: the attention reads it as one key (and value) of `padded` values.
+// With q_rank > 0 the same row of x holds, `q_rank` values before x's start, a second vector (the query's latent) that is
+// normed with its own weight into q_out: both norms of a token in one launch.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_norm_rope_cache_write_kernel(const T* __restrict__ x, long long x_stride,
                                                                            const float* __restrict__ w, T* __restrict__ cache,
@@ -48,15 +63,27 @@ __global__ void __launch_bounds__(128) latent_norm_rope_cache_write_kernel(const
                                                                            const int* __restrict__ token_seq,
                                                                            const int* __restrict__ block_table, int max_blocks,
                                                                            int block_size, int rank, int padded, float eps,
-                                                                           int rot_dim, int rot_n, const float* __restrict__ inv_freq,
+                                                                           int rot_dim, PartRotation rot, int q_rank,
+                                                                           const float* __restrict__ wq, T* __restrict__ q_out,
                                                                            int* __restrict__ error_flag) {
   __shared__ float scratch[33];
+  pdl_launch_dependents();
+  pdl_wait();
   const int t = blockIdx.x;
   const T* xr = x + (size_t)t * x_stride;
+  if (q_rank > 0) {
+    const T* qr = xr - q_rank;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_f32(qr[i]); sq = fmaf(v, v, sq); }
+    sq = block_sum(sq, scratch);
+    const float inv_q = 1.0f / sqrtf(sq / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) q_out[(size_t)t * q_rank + i] = from_f32<T>((to_f32(qr[i]) * inv_q) * wq[i]);
+  }
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_f32(xr[i]); ss = fmaf(v, v, ss); }
   ss = block_sum(ss, scratch);
   const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
+  if (cache == nullptr) return;
   const int pos = positions[t];
   const int blk = pos / block_size;
   const int page = blk < max_blocks ? block_table[(size_t)token_seq[t] * max_blocks + blk] : -1;
@@ -66,15 +93,15 @@ __global__ void __launch_bounds__(128) latent_norm_rope_cache_write_kernel(const
   }
   T* dst = cache + (size_t)page * page_stride + (size_t)(pos % block_size) * padded;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<T>((to_f32(xr[i]) * inv) * w[i]);
-  const int half = rot_n / 2;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+  for (int i = threadIdx.x; i < rot.n / 2; i += blockDim.x) {
     float sn, cs;
-    sincosf((float)pos * inv_freq[i], &sn, &cs);
-    const float u = to_f32(xr[rank + i]), v = to_f32(xr[rank + half + i]);
-    dst[rank + i] = from_f32<T>(rot_first(u, v, cs, sn));
-    dst[rank + half + i] = from_f32<T>(rot_second(u, v, cs, sn));
+    rot.angle(pos, i, &cs, &sn);
+    const int a = rank + rot.first(i), b = rank + rot.second(i);
+    const float u = to_f32(xr[a]), v = to_f32(xr[b]);
+    dst[a] = from_f32<T>(rot_first(u, v, cs, sn));
+    dst[b] = from_f32<T>(rot_second(u, v, cs, sn));
   }
-  for (int i = rank + rot_n + threadIdx.x; i < padded; i += blockDim.x)
+  for (int i = rank + rot.n + threadIdx.x; i < padded; i += blockDim.x)
     dst[i] = i < rank + rot_dim ? xr[i] : from_f32<T>(0.f);
 }
 
@@ -83,13 +110,13 @@ __global__ void __launch_bounds__(128) latent_norm_rope_cache_write_kernel(const
 template <typename T>
 __global__ void __launch_bounds__(128) latent_query_rope_kernel(const T* __restrict__ q, long long q_stride, T* __restrict__ qa,
                                                                 long long qa_stride, const int* __restrict__ positions,
-                                                                int heads, int plain, int rot_dim, int rot_n,
-                                                                const float* __restrict__ inv_freq, int rank, int padded) {
+                                                                int heads, int plain, int rot_dim, PartRotation rot, int rank,
+                                                                int padded) {
   extern __shared__ float cs_sn[];                // cos[half], sin[half]
   const int t = blockIdx.x;
   const int pos = positions[t];
-  const int half = rot_n / 2;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &cs_sn[half + i], &cs_sn[i]);
+  const int half = rot.n / 2;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) rot.angle(pos, i, &cs_sn[i], &cs_sn[half + i]);
   __syncthreads();
   const int tail = padded - rank;                 // values behind the expanded part of a head of qa
   const int width = plain + rot_dim;
@@ -97,10 +124,11 @@ __global__ void __launch_bounds__(128) latent_query_rope_kernel(const T* __restr
     const int h = j / tail, i = j % tail;
     const T* src = q + (size_t)t * q_stride + (size_t)h * width + plain;
     float o = 0.f;
-    if (i < rot_n) {
-      const int p = i < half ? i : i - half;
-      const float u = to_f32(src[p]), v = to_f32(src[p + half]);
-      o = i < half ? rot_first(u, v, cs_sn[p], cs_sn[half + p]) : rot_second(u, v, cs_sn[p], cs_sn[half + p]);
+    if (i < rot.n) {
+      const int p = rot.interleaved ? i >> 1 : (i < half ? i : i - half);
+      const bool is_first = rot.interleaved ? (i & 1) == 0 : i < half;
+      const float u = to_f32(src[rot.first(p)]), v = to_f32(src[rot.second(p)]);
+      o = is_first ? rot_first(u, v, cs_sn[p], cs_sn[half + p]) : rot_second(u, v, cs_sn[p], cs_sn[half + p]);
     } else if (i < rot_dim) {
       o = to_f32(src[i]);
     }
@@ -233,36 +261,41 @@ LMSF_API int lmsf_latent_norm_cache_write(const void* x, long long x_stride, con
 }
 
 // x: rows of [n, rank + rot_dim] of `dtype`; inv_freq: float32 [rot_n / 2]; cache: [pages, 1, 1, block_size, padded] with
-// padded >= rank + rot_dim.
+// padded >= rank + rot_dim, or null (nothing is cached).  interleaved: neighbours are paired, else halves; rot_mult multiplies
+// cos and sin.  q_rank > 0: x[t] is preceded in memory by q_rank values of a second vector, normed with wq (float32 [q_rank])
+// into q_out ([n, q_rank] of `dtype`).
 LMSF_API int lmsf_latent_norm_rope_cache_write(const void* x, long long x_stride, const float* w, void* cache,
                                                long long page_stride, const int* positions, const int* token_seq,
                                                const int* block_table, int max_blocks, int block_size, int n, int rank,
-                                               int padded, float eps, int rot_dim, int rot_n, const float* inv_freq, int dtype,
-                                               int* error_flag, void* stream) {
+                                               int padded, float eps, int rot_dim, int rot_n, const float* inv_freq,
+                                               int interleaved, float rot_mult, int q_rank, const float* wq, void* q_out,
+                                               int dtype, int* error_flag, void* stream) {
   using namespace lmsf;
   if (n <= 0) return 0;
   if (rank <= 0 || rot_dim < 0 || padded < rank + rot_dim || block_size <= 0 || max_blocks <= 0 || !(eps > 0.f))
     LMSF_REFUSE("latent cache: rank=%d rot_dim=%d padded=%d block_size=%d max_blocks=%d", rank, rot_dim, padded, block_size, max_blocks);
   if (rot_n < 0 || rot_n % 2 || rot_n > rot_dim || (rot_n > 0 && !inv_freq))
     LMSF_REFUSE("latent cache: %d rotated values of %d (even, with their frequencies)", rot_n, rot_dim);
+  if (q_rank < 0 || (q_rank > 0 && (!wq || !q_out || x_stride < q_rank + rank + rot_dim)))
+    LMSF_REFUSE("latent cache: a second vector of %d values needs its weight, its output and its place before x", q_rank);
   cudaStream_t s = (cudaStream_t)stream;
+  const PartRotation rot{inv_freq, rot_n, interleaved ? 1 : 0, rot_mult};
   if (dtype == LMSF_F32)
-    latent_norm_rope_cache_write_kernel<float><<<n, 128, 0, s>>>((const float*)x, x_stride, w, (float*)cache, page_stride, positions,
-                                                                 token_seq, block_table, max_blocks, block_size, rank, padded, eps,
-                                                                 rot_dim, rot_n, inv_freq, error_flag);
-  else if (dtype == LMSF_BF16)
-    latent_norm_rope_cache_write_kernel<bf16><<<n, 128, 0, s>>>((const bf16*)x, x_stride, w, (bf16*)cache, page_stride, positions,
-                                                                token_seq, block_table, max_blocks, block_size, rank, padded, eps,
-                                                                rot_dim, rot_n, inv_freq, error_flag);
-  else LMSF_REFUSE("latent cache: unknown dtype code %d", dtype);
-  return LMSF_LAUNCH_STATUS();
+    return launch_pdl(latent_norm_rope_cache_write_kernel<float>, dim3(n), dim3(128), 0, s, (const float*)x, x_stride, w,
+                      (float*)cache, page_stride, positions, token_seq, block_table, max_blocks, block_size, rank, padded, eps,
+                      rot_dim, rot, q_rank, wq, (float*)q_out, error_flag);
+  if (dtype == LMSF_BF16)
+    return launch_pdl(latent_norm_rope_cache_write_kernel<bf16>, dim3(n), dim3(128), 0, s, (const bf16*)x, x_stride, w,
+                      (bf16*)cache, page_stride, positions, token_seq, block_table, max_blocks, block_size, rank, padded, eps,
+                      rot_dim, rot, q_rank, wq, (bf16*)q_out, error_flag);
+  LMSF_REFUSE("latent cache: unknown dtype code %d", dtype);
 }
 
 // q: [n, heads * (plain + rot_dim)] of `dtype`; qa: [n, heads * padded] of `dtype`, of which this call writes the columns
-// rank .. padded of every head.
+// rank .. padded of every head.  interleaved, rot_mult: as above.
 LMSF_API int lmsf_latent_query_rope(const void* q, long long q_stride, void* qa, long long qa_stride, const int* positions,
-                                    int n, int heads, int plain, int rot_dim, int rot_n, const float* inv_freq, int rank,
-                                    int padded, int dtype, void* stream) {
+                                    int n, int heads, int plain, int rot_dim, int rot_n, const float* inv_freq, int interleaved,
+                                    float rot_mult, int rank, int padded, int dtype, void* stream) {
   using namespace lmsf;
   if (n <= 0) return 0;
   if (heads <= 0 || plain < 0 || rot_dim < 0 || rank <= 0 || padded < rank + rot_dim)
@@ -272,12 +305,13 @@ LMSF_API int lmsf_latent_query_rope(const void* q, long long q_stride, void* qa,
   if (padded == rank) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const size_t smem = (size_t)rot_n * sizeof(float);
+  const PartRotation rot{inv_freq, rot_n, interleaved ? 1 : 0, rot_mult};
   if (dtype == LMSF_F32)
     latent_query_rope_kernel<float><<<n, 128, smem, s>>>((const float*)q, q_stride, (float*)qa, qa_stride, positions, heads, plain,
-                                                         rot_dim, rot_n, inv_freq, rank, padded);
+                                                         rot_dim, rot, rank, padded);
   else if (dtype == LMSF_BF16)
     latent_query_rope_kernel<bf16><<<n, 128, smem, s>>>((const bf16*)q, q_stride, (bf16*)qa, qa_stride, positions, heads, plain,
-                                                        rot_dim, rot_n, inv_freq, rank, padded);
+                                                        rot_dim, rot, rank, padded);
   else LMSF_REFUSE("latent query: unknown dtype code %d", dtype);
   return LMSF_LAUNCH_STATUS();
 }

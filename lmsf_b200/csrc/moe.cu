@@ -388,6 +388,22 @@ __global__ void relu2_kernel(T* __restrict__ x, long long n) {
   if (i < n) { const float r = fmaxf(to_f32(x[i]), 0.f); x[i] = from_f32<T>(r * r); }
 }
 
+// the same on bfloat16 with 16 bytes a thread: counts that 8 divides, a 16-byte aligned pointer
+__global__ void relu2_8_kernel(bf16* __restrict__ x, long long n8) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  uint4 v = reinterpret_cast<uint4*>(x)[i];
+  __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    float2 f = __bfloat1622float2(p[k]);
+    f.x = fmaxf(f.x, 0.f);
+    f.y = fmaxf(f.y, 0.f);
+    p[k] = __floats2bfloat162_rn(f.x * f.x, f.y * f.y);
+  }
+  reinterpret_cast<uint4*>(x)[i] = v;
+}
+
 }  // namespace lmsf
 
 LMSF_API int lmsf_moe_topk(const float* logits, long long ld, const float* bias, int n, int experts, int top, int* ids,
@@ -491,7 +507,9 @@ LMSF_API int lmsf_relu2(void* x, long long n, int dtype, void* stream) {
   if (n <= 0) return 0;
   const unsigned blocks = (unsigned)((n + 255) / 256);
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == LMSF_F32) relu2_kernel<float><<<blocks, 256, 0, s>>>((float*)x, n);
+  if (dtype == LMSF_BF16 && n % 8 == 0 && (uintptr_t)x % 16 == 0)
+    relu2_8_kernel<<<(unsigned)((n / 8 + 255) / 256), 256, 0, s>>>((bf16*)x, n / 8);
+  else if (dtype == LMSF_F32) relu2_kernel<float><<<blocks, 256, 0, s>>>((float*)x, n);
   else if (dtype == LMSF_BF16) relu2_kernel<bf16><<<blocks, 256, 0, s>>>((bf16*)x, n);
   else LMSF_REFUSE("relu2: unknown dtype code %d", dtype);
   return LMSF_LAUNCH_STATUS();

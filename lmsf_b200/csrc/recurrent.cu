@@ -368,7 +368,7 @@ template <typename T, bool BLOCK>
 __global__ void grouped_gated_norm_kernel(T* __restrict__ out, long long out_stride, const float* __restrict__ x,
                                           long long x_stride, const T* __restrict__ gate, long long gate_stride,
                                           const float* __restrict__ w, int wlen, int n, int n_groups, int gsize, float eps,
-                                          int gate_silu, int gate_first) {
+                                          int gate_silu, int gate_first, float out_scale) {
   __shared__ float scratch[33];
   const int team = BLOCK ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int me = BLOCK ? threadIdx.x : (threadIdx.x & 31), step = BLOCK ? blockDim.x : 32;
@@ -392,7 +392,7 @@ __global__ void grouped_gated_norm_kernel(T* __restrict__ out, long long out_str
     if (gate_first) v *= gv;
     v = (v * inv) * w[(grp * gsize + i) % wlen];
     if (!gate_first) v *= gv;
-    o[i] = from_f32<T>(v);
+    o[i] = from_f32<T>(v * out_scale);
   }
 }
 
@@ -405,7 +405,7 @@ template <typename T, bool BLOCK, int PER, int V>
 __global__ void __launch_bounds__(BLOCK ? 256 : 128) grouped_gated_norm_reg_kernel(
     T* __restrict__ out, long long out_stride, const float* __restrict__ x, long long x_stride, const T* __restrict__ gate,
     long long gate_stride, const float* __restrict__ w, int wlen, int n, int n_groups, int gsize, float eps, int gate_silu,
-    int gate_first) {
+    int gate_first, float out_scale) {
   __shared__ float scratch[33];
   const int team = BLOCK ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int me = BLOCK ? threadIdx.x : (threadIdx.x & 31), step = BLOCK ? 256 : 32;
@@ -448,7 +448,7 @@ __global__ void __launch_bounds__(BLOCK ? 256 : 128) grouped_gated_norm_reg_kern
       for (int e = 0; e < V; ++e) {
         float r = (v[j][e] * inv) * w[wi + e];
         if (!gate_first) r *= gv[j][e];
-        ov.v[e] = from_f32<T>(r);
+        ov.v[e] = from_f32<T>(r * out_scale);
       }
       *reinterpret_cast<NormVec<T, V>*>(o + i) = ov;
     }
@@ -517,9 +517,10 @@ LMSF_API int lmsf_gated_scan(float* out, long long out_stride, const void* q, co
 }
 
 // x: float32 [n, n_groups * gsize]; gate (may be null) and out: rows of `dtype`; w: float32 [wlen], wlen divides into the row.
+// out_scale multiplies the result before it is rounded.
 LMSF_API int lmsf_grouped_gated_norm(void* out, long long out_stride, const float* x, long long x_stride, const void* gate,
                                      long long gate_stride, const float* w, int wlen, int n, int n_groups, int gsize, float eps,
-                                     int gate_silu, int gate_first, int dtype, void* stream) {
+                                     int gate_silu, int gate_first, float out_scale, int dtype, void* stream) {
   using namespace lmsf;
   if (n <= 0) return 0;
   if (n_groups <= 0 || gsize <= 0 || wlen <= 0 || !(eps > 0.f)) LMSF_REFUSE("grouped_gated_norm: %d groups of %d, eps %g", n_groups, gsize, eps);
@@ -531,7 +532,7 @@ LMSF_API int lmsf_grouped_gated_norm(void* out, long long out_stride, const floa
   const bool wide = gsize % 4 == 0 && wlen % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && (!gate || gate_stride % 4 == 0) &&
                     ((uintptr_t)x | (uintptr_t)w) % 16 == 0 && ((uintptr_t)out | (uintptr_t)gate) % (4 * esz) == 0;
   const int per = ceil_div(gsize, (block ? 256 : 32) * (wide ? 4 : 1));
-#define LMSF_REG(T, B, P, V) grouped_gated_norm_reg_kernel<T, B, P, V><<<blocks, B ? 256 : 128, 0, s>>>((T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first)
+#define LMSF_REG(T, B, P, V) grouped_gated_norm_reg_kernel<T, B, P, V><<<blocks, B ? 256 : 128, 0, s>>>((T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first, out_scale)
 #define LMSF_CASE(T, B, P) if (per <= P) { if (wide) LMSF_REG(T, B, P, 4); else LMSF_REG(T, B, P, 1); return LMSF_LAUNCH_STATUS(); }
 #define LMSF_NARROW(T, B, P) if (!wide && per <= P) { LMSF_REG(T, B, P, 1); return LMSF_LAUNCH_STATUS(); }
 #define LMSF_PICK(T)                                                                          \
@@ -544,7 +545,7 @@ LMSF_API int lmsf_grouped_gated_norm(void* out, long long out_stride, const floa
 #undef LMSF_NARROW
 #undef LMSF_CASE
 #undef LMSF_REG
-#define LMSF_GO(T, B) grouped_gated_norm_kernel<T, B><<<blocks, B ? 256 : 128, 0, s>>>((T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first)
+#define LMSF_GO(T, B) grouped_gated_norm_kernel<T, B><<<blocks, B ? 256 : 128, 0, s>>>((T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first, out_scale)
   if (dtype == LMSF_F32) { if (block) LMSF_GO(float, true); else LMSF_GO(float, false); }
   else if (dtype == LMSF_BF16) { if (block) LMSF_GO(bf16, true); else LMSF_GO(bf16, false); }
   else LMSF_REFUSE("grouped_gated_norm: unknown dtype code %d", dtype);

@@ -6,7 +6,8 @@
 // looked up in the request's block table here rather than through a precomputed slot mapping; k
 // goes to the cache only (attention always reads keys from pages).
 //
-// Cache layout of one layer: [page][2 (k, v)][kv_head][slot][head_dim].
+// Cache layout of one layer: [page][2 (k, v)][kv_head][slot][head_dim]; without v (a cache whose keys are its values):
+// [page][1][kv_head][slot][head_dim].
 #include "common.cuh"
 #include <type_traits>
 
@@ -98,6 +99,7 @@ __global__ void rope_cache_kernel(RopeCacheArgs a) {
     const int g = w / tail, i = rot + w % tail;
     kc[g * head_pitch + i] = k[(size_t)g * hd + i];
   }
+  if (!a.v) return;
   for (int w = threadIdx.x; w < a.n_kv_heads * hd; w += blockDim.x) {
     const int g = w / hd, i = w % hd;
     vc[g * head_pitch + i] = v[(size_t)g * hd + i];
@@ -142,7 +144,7 @@ __global__ void rope_cache_vec_kernel(RopeCacheArgs a) {
   const int n_qrot = a.n_q_heads * hv;
   const int n_krot = kc ? a.n_kv_heads * hv : 0;
   const int n_ktail = kc ? a.n_kv_heads * tail_v : 0;
-  const int n_v = kc ? a.n_kv_heads * hd_v : 0;
+  const int n_v = (kc && a.v) ? a.n_kv_heads * hd_v : 0;
   const int total = n_qrot + n_krot + n_ktail + n_v;
   typedef typename std::conditional<VEC == 8, uint4, float4>::type Raw;
   for (int w = blockIdx.y * blockDim.x + threadIdx.x; w < total; w += gridDim.y * blockDim.x) {
@@ -189,8 +191,8 @@ LMSF_API int lmsf_rope_cache_write(void* q, const void* k, const void* v, long l
   if (head_dim <= 0 || n_q_heads < 0 || n_kv_heads < 0) LMSF_REFUSE("rope_cache: bad head sizes");
   if (inv_freq && (rot_dim <= 0 || rot_dim % 2 || rot_dim > head_dim))
     LMSF_REFUSE("rope_cache: rot_dim=%d must be even and at most head_dim=%d", rot_dim, head_dim);
-  if (cache && (!k || !v || !block_table || !token_seq || block_size <= 0 || max_blocks <= 0))
-    LMSF_REFUSE("rope_cache: a cache write needs k, v, a block table and the block size");
+  if (cache && (!k || !block_table || !token_seq || block_size <= 0 || max_blocks <= 0))
+    LMSF_REFUSE("rope_cache: a cache write needs k, a block table and the block size");
   if (dtype != LMSF_F32 && dtype != LMSF_BF16) LMSF_REFUSE("rope_cache: unknown dtype code %d", dtype);
   RopeCacheArgs a{q, k, v, q_stride, k_stride, v_stride, positions, token_seq, block_table, max_blocks, block_size,
                   cache, page_stride, inv_freq, rot_dim, is_neox, n_q_heads, n_kv_heads, head_dim, error_flag};
@@ -202,7 +204,7 @@ LMSF_API int lmsf_rope_cache_write(void* q, const void* k, const void* v, long l
                       q_stride % vec == 0 && (!cache || (k_stride % vec == 0 && v_stride % vec == 0 && page_stride % vec == 0)) &&
                       ((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)cache) % 16 == 0;
   if (vec_ok) {
-    const int items = (n_q_heads * (rot / 2) + (cache ? n_kv_heads * (rot / 2 + (head_dim - rot) + head_dim) : 0)) / vec;
+    const int items = (n_q_heads * (rot / 2) + (cache ? n_kv_heads * (rot / 2 + (head_dim - rot) + (v ? head_dim : 0)) : 0)) / vec;
     int gy = ceil_div(items > 0 ? items : 1, 128);
     if (gy > 8) gy = 8;
     // Every block of a token computes the token's angles and looks its page up before it moves a byte: with many

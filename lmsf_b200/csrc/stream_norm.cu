@@ -258,6 +258,67 @@ __global__ void __launch_bounds__(kThreads) gated_branches_kernel(float* __restr
   }
 }
 
+// Two branches of the same stream that are added together, and the two norms of the sum that the next block's branches read:
+//   res <- res + c1 * y1 + c2 * y2  (either may be null);  h1 = norm(res) * w1;  h2 = norm(res) * w2  (either may be null)
+// The root of the mean square is taken once (one eps for both).  float32 inside; one block per token.
+template <typename T, int PER, int V>
+__global__ void __launch_bounds__(kThreads) stream_branches_kernel(float* __restrict__ res, const T* __restrict__ y1, float c1,
+                                                                   const T* __restrict__ y2, float c2, T* __restrict__ h1,
+                                                                   const float* __restrict__ w1, T* __restrict__ h2,
+                                                                   const float* __restrict__ w2, int hidden, float eps) {
+  __shared__ float scratch[33];
+  const size_t base = (size_t)blockIdx.x * hidden;
+  float r[PER][V];
+  pdl_launch_dependents();
+  pdl_wait();
+  float ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < PER; ++it) {
+    const int i = (it * kThreads + threadIdx.x) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) r[it][e] = 0.f;
+    if (i < hidden) {
+      float y[V];
+      ld_vec<V>(res + base + i, r[it]);
+      if (y1 != nullptr) {
+        ld_vec<V>(y1 + base + i, y);
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[it][e] = fmaf(c1, y[e], r[it][e]);
+      }
+      if (y2 != nullptr) {
+        ld_vec<V>(y2 + base + i, y);
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[it][e] = fmaf(c2, y[e], r[it][e]);
+      }
+      if (y1 != nullptr || y2 != nullptr) st_vec<V>(res + base + i, r[it]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(r[it][e], r[it][e], ss);
+  }
+  if (h1 == nullptr && h2 == nullptr) return;
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+  for (int it = 0; it < PER; ++it) {
+    const int i = (it * kThreads + threadIdx.x) * V;
+    if (i < hidden) {
+      float w[V], o[V];
+      if (h1 != nullptr) {
+        ld_vec<V>(w1 + i, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = (r[it][e] * inv) * w[e];
+        st_vec<V>(h1 + base + i, o);
+      }
+      if (h2 != nullptr) {
+        ld_vec<V>(w2 + i, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = (r[it][e] * inv) * w[e];
+        st_vec<V>(h2 + base + i, o);
+      }
+    }
+  }
+}
+
 // out[t] = [a[t] | b[t]] in the activation type: two float32 streams side by side as the input of one product.
 template <typename T>
 __global__ void stream_concat_kernel(T* __restrict__ out, const float* __restrict__ a, const float* __restrict__ b,
@@ -289,6 +350,22 @@ __global__ void stream_concat4_kernel(T* __restrict__ out, const float* __restri
     packed.y = *reinterpret_cast<unsigned*>(&hi);
     *reinterpret_cast<uint2*>(dst) = packed;
   }
+}
+
+template <typename T>
+static int pick_branches(float* res, const void* y1, float c1, const void* y2, float c2, void* h1, const float* w1, void* h2,
+                         const float* w2, int n, int hidden, float eps, cudaStream_t s) {
+  const bool wide = hidden % 4 == 0 && ((uintptr_t)res | (uintptr_t)w1 | (uintptr_t)w2) % 16 == 0 &&
+                    ((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)h1 | (uintptr_t)h2) % (4 * sizeof(T)) == 0;
+  const int per = ceil_div(hidden, kThreads * (wide ? 4 : 1));
+#define LMSF_GO(P, V) return launch_pdl(stream_branches_kernel<T, P, V>, dim3(n), dim3(kThreads), 0, s, res, (const T*)y1, c1, \
+                                        (const T*)y2, c2, (T*)h1, w1, (T*)h2, w2, hidden, eps)
+#define LMSF_CASE(P) if (per <= P) { if (wide) LMSF_GO(P, 4); else LMSF_GO(P, 1); }
+  LMSF_CASE(1) LMSF_CASE(2) LMSF_CASE(4) LMSF_CASE(8) LMSF_CASE(16)
+  if (!wide) { if (per <= 32) LMSF_GO(32, 1); LMSF_GO(64, 1); }
+#undef LMSF_CASE
+#undef LMSF_GO
+  return LMSF_EBADARG;
 }
 
 template <typename T, int PER, int V>
@@ -379,6 +456,20 @@ LMSF_API int lmsf_gated_branches(float* res, const float* z, long long ldz, cons
   if (dtype == LMSF_F32) return pick_gated<float>(res, z, ldz, b, y1, y2, h, w_next, n, hidden, eps_next, s);
   if (dtype == LMSF_BF16) return pick_gated<bf16>(res, z, ldz, b, y1, y2, h, w_next, n, hidden, eps_next, s);
   LMSF_REFUSE("gated_branches: unknown dtype code %d", dtype);
+}
+
+// res: float32 [n, hidden]; y1, y2, h1, h2 (each may be null): [n, hidden] of `dtype`; w1, w2: float32 [hidden] for the h that is
+// asked for.
+LMSF_API int lmsf_stream_branches(float* res, const void* y1, float c1, const void* y2, float c2, void* h1, const float* w1,
+                                  void* h2, const float* w2, int n, int hidden, float eps, int dtype, void* stream) {
+  using namespace lmsf;
+  if (n <= 0) return 0;
+  if (hidden <= 0 || hidden > kThreads * kMaxPerThread) LMSF_REFUSE("stream_branches: width %d is outside 1..%d", hidden, kThreads * kMaxPerThread);
+  if ((h1 && !w1) || (h2 && !w2) || ((h1 || h2) && !(eps > 0.f))) LMSF_REFUSE("stream_branches: a norm needs its weight and a positive eps");
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == LMSF_F32) return pick_branches<float>(res, y1, c1, y2, c2, h1, w1, h2, w2, n, hidden, eps, s);
+  if (dtype == LMSF_BF16) return pick_branches<bf16>(res, y1, c1, y2, c2, h1, w1, h2, w2, n, hidden, eps, s);
+  LMSF_REFUSE("stream_branches: unknown dtype code %d", dtype);
 }
 
 // out: [n, 2 * hidden] of `dtype` = [a | b], both float32 [n, hidden].

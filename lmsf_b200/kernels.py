@@ -121,6 +121,19 @@ def embedding(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, error_f
     _check(rc, "embedding.cu", "lmsf_embedding")
 
 
+def embedding_stream(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0,
+                     error_flag: Optional[torch.Tensor] = None):
+    """out[t] = table[ids[t]] * scale in float32 (not rounded, whatever the table's type): the start of a residual stream."""
+    n, hidden = out.shape
+    if out.dtype != torch.float32 or not out.is_contiguous() or table.shape[1] != hidden or not table.is_contiguous():
+        raise KernelError("embedding_stream: out float32 [n, hidden] and a contiguous table [vocab, hidden]")
+    f = _func("embedding.cu", "lmsf_embedding_stream",
+              [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p])
+    rc = f(_ptr(out), _ptr(table), _i32(ids, "ids"), n, hidden, table.shape[0], float(scale), dtype_code(table.dtype),
+           _i32(error_flag, "error_flag"), _stream())
+    _check(rc, "embedding.cu", "lmsf_embedding")
+
+
 def embedding_pairs(out: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor,
                     token_seq: torch.Tensor, cu_q: torch.Tensor, state_slot: torch.Tensor, last: torch.Tensor, buckets: int,
                     mul_prev: int, mul_cur: int, scale: float = 1.0, error_flag: Optional[torch.Tensor] = None):
@@ -193,7 +206,8 @@ def rope_cache_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[tor
                      n_q_heads: int, n_kv_heads: int, head_dim: int, error_flag: Optional[torch.Tensor] = None):
     """Rotates q in place; writes rotated k and v into `cache` [pages, 2, n_kv_heads, block_size, head_dim]
     at the page that `block_table[token_seq[t], positions[t] // block_size]` names.  q, k, v: [n, heads*head_dim]
-    views whose last dimension is contiguous (row strides are free).  cache None: q only."""
+    views whose last dimension is contiguous (row strides are free).  cache None: q only.  v None with a cache: k alone is
+    written, into [pages, 1, n_kv_heads, block_size, head_dim] (a cache whose keys are its values)."""
     n = q.shape[0]
     for name, t, heads in (("q", q, n_q_heads), ("k", k, n_kv_heads), ("v", v, n_kv_heads)):
         if t is None:
@@ -205,9 +219,10 @@ def rope_cache_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[tor
     page_stride = 0
     max_blocks = 0
     if cache is not None:
-        if cache.dtype != q.dtype or not cache.is_contiguous() or tuple(cache.shape[1:]) != (2, n_kv_heads, block_size, head_dim):
+        planes = 2 if v is not None else 1
+        if cache.dtype != q.dtype or not cache.is_contiguous() or tuple(cache.shape[1:]) != (planes, n_kv_heads, block_size, head_dim):
             raise KernelError(f"rope_cache: cache of shape {tuple(cache.shape)} does not match "
-                              f"[pages, 2, {n_kv_heads}, {block_size}, {head_dim}] of {q.dtype}")
+                              f"[pages, {planes}, {n_kv_heads}, {block_size}, {head_dim}] of {q.dtype}")
         page_stride = cache.stride(0)
         max_blocks = block_table.shape[1]
     if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dim // 2):
@@ -278,6 +293,17 @@ _GENERIC_MASKED_ARGS = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_
 _GENERIC_WEIGHTS_ARGS = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p,
                          c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                          c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]
+_GENERIC_DIST_ARGS = _GENERIC_WEIGHTS_ARGS[:-1] + [c_void_p, c_int, c_void_p]
+
+
+def _dist_args(dist: Optional[torch.Tensor], heads: int) -> Tuple[Optional[int], int]:
+    """A table of what is added to the scores by distance, float32 [n_q_heads, entries] (the last entry serves every larger
+    distance) -> (pointer, entries)."""
+    if dist is None:
+        return None, 0
+    if dist.dtype != torch.float32 or dist.dim() != 2 or dist.shape[0] != heads or dist.shape[1] < 1 or not dist.is_contiguous():
+        raise KernelError("attention: a table of distances must be contiguous float32 [n_q_heads, entries]")
+    return _ptr(dist), dist.shape[1]
 
 
 def attention_generic(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
@@ -286,7 +312,7 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, b
                       slopes: Optional[torch.Tensor] = None, chunk: int = 0,
                       log_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, sinks: Optional[torch.Tensor] = None,
                       gate: Optional[torch.Tensor] = None, keep_first: int = 0, sigmoid: bool = False,
-                      head_bias: Optional[torch.Tensor] = None):
+                      head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None, kv_planes: int = 2):
     """out[t] = softmax(scale q[t] K^T) V over the keys lo..positions[t] of token t's request, read from pages.
     q, out: [n, n_q_heads * head_dim] (last dimension contiguous); window <= 0 means all keys; softcap > 0 caps the
     scaled scores smoothly, softcap * tanh(score / softcap); slopes (float32 [n_q_heads]) adds
@@ -295,12 +321,14 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, b
     scaled scores.  sinks (float32 [n_q_heads]): exp(sink) is one more term of the softmax's denominator.  gate ([n,
     n_q_heads] view of q's dtype): head h's output is multiplied by sigmoid(gate[t, h]).  keep_first (with a window): the
     request's first keep_first keys stay visible behind the window.  sigmoid: a visible key's weight is sigmoid(score), not
-    normalised over the keys.  head_bias (float32 [n_q_heads]): added to every scaled score of its head."""
+    normalised over the keys.  head_bias (float32 [n_q_heads]): added to every scaled score of its head.  dist (float32
+    [n_q_heads, entries]): entry min(query position - key position, entries - 1) of the head's row is added to the scaled
+    score.  kv_planes 1: the cache holds one vector per token and kv head that is key and value at once."""
     n = q.shape[0]
     if q.stride(1) != 1 or out.stride(1) != 1 or q.shape[1] != n_q_heads * head_dim or out.shape != q.shape:
         raise KernelError("attention: q and out must be [n, heads * head_dim] with a contiguous last dimension")
     if cache.dtype != q.dtype or out.dtype != q.dtype or not cache.is_contiguous() or \
-            tuple(cache.shape[1:]) != (2, n_kv_heads, block_size, head_dim):
+            kv_planes not in (1, 2) or tuple(cache.shape[1:]) != (kv_planes, n_kv_heads, block_size, head_dim):
         raise KernelError(f"attention: cache of shape {tuple(cache.shape)} / {cache.dtype} does not match the heads")
     _per_head(slopes, n_q_heads, "slopes")
     _per_head(sinks, n_q_heads, "sinks")
@@ -310,12 +338,13 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, b
     _per_head(r2, n_q_heads, "the logarithmic bias")
     if gate is not None and (gate.shape != (n, n_q_heads) or gate.stride(1) != 1 or gate.dtype != q.dtype):
         raise KernelError("attention: the gate must be [n, heads] of q's dtype")
-    f = _func("attention_generic.cu", "lmsf_attention_generic_weights", _GENERIC_WEIGHTS_ARGS)
+    f = _func("attention_generic.cu", "lmsf_attention_generic_dist", _GENERIC_DIST_ARGS)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0),
            _i32(block_table, "block_table"), block_table.shape[1], block_size, _i32(token_seq, "token_seq"),
            _i32(positions, "positions"), float(scale), float(softcap or 0.0), _ptr(slopes), int(window or 0), n, n_q_heads,
-           n_kv_heads, head_dim, dtype_code(q.dtype), 0, _ptr(gate), gate.stride(0) if gate is not None else 0,
-           int(chunk or 0), _ptr(r1), _ptr(r2), _ptr(sinks), int(keep_first or 0), 1 if sigmoid else 0, _ptr(head_bias), _stream())
+           n_kv_heads, head_dim, dtype_code(q.dtype), int(kv_planes == 1), _ptr(gate), gate.stride(0) if gate is not None else 0,
+           int(chunk or 0), _ptr(r1), _ptr(r2), _ptr(sinks), int(keep_first or 0), 1 if sigmoid else 0, _ptr(head_bias),
+           *_dist_args(dist, n_q_heads), _stream())
     _check(rc, "attention_generic.cu", "lmsf_attention_generic")
 
 
@@ -433,11 +462,18 @@ def _prenorm_args(prenorm, M: int, what: str):
     return _ptr(sumsq), sumsq.shape[1], sumsq.stride(0), float(eps), int(width)
 
 
-def gemm_skinny(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, fuse_act: Optional[str] = None, prenorm=None):
+def _bf16_bias(bias: Optional[torch.Tensor], n: int, what: str) -> None:
+    if bias is not None and (bias.dtype != torch.bfloat16 or bias.shape != (n,) or not bias.is_contiguous()):
+        raise KernelError(f"{what}: the bias must be contiguous bfloat16 [{n}]")
+
+
+def gemm_skinny(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, fuse_act: Optional[str] = None, prenorm=None,
+                bias: Optional[torch.Tensor] = None, act: Optional[str] = None):
     """out[M, N] = x[M, K] w[N, K]^T for M <= 16 (bfloat16 in, bfloat16 or float32 out).  With fuse_act
     ("silu", "gelu_tanh") w is [2 N_out, K] (gate rows, then up rows) and out[M, N_out] = act(x gate^T) * (x up^T).
     prenorm = (sumsq, eps, width): x is a residual stream times a norm weight and the sums of row m are multiplied by
-    1 / sqrt(sum(sumsq[m]) / width + eps) first (what `gemm_skinny_residual` leaves)."""
+    1 / sqrt(sum(sumsq[m]) / width + eps) first (what `gemm_skinny_residual` leaves).  bias (bfloat16 [N]) is added to the
+    sums; act "relu2": the square of max(sum, 0) (both without fuse_act)."""
     M, K = x.shape
     N = w.shape[0]
     n_out = N // 2 if fuse_act else N
@@ -447,12 +483,15 @@ def gemm_skinny(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, fuse_act: O
         raise KernelError("gemm_skinny: out must be bfloat16 or float32")
     if fuse_act is not None and fuse_act not in ACT_CODES:
         raise KernelError(f"gemm_skinny: unknown activation {fuse_act!r}")
+    if act not in (None, "relu2"):
+        raise KernelError(f"gemm_skinny: unknown activation {act!r} of the plain form")
+    _bf16_bias(bias, N, "gemm_skinny")
     f = _func("gemm_skinny.cu", "lmsf_gemm_skinny",
               [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_int,
-               c_void_p, c_int, c_longlong, c_float, c_int, c_void_p], SKINNY_DEFINES)
+               c_void_p, c_int, c_longlong, c_float, c_int, c_void_p, c_int, c_void_p], SKINNY_DEFINES)
     rc = f(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
            ACT_CODES[fuse_act] if fuse_act else -1, int(out.dtype == torch.float32),
-           *_prenorm_args(prenorm, M, "gemm_skinny"), _stream())
+           *_prenorm_args(prenorm, M, "gemm_skinny"), _ptr(bias), int(act == "relu2"), _stream())
     _check(rc, "gemm_skinny.cu", "lmsf_gemm_skinny", SKINNY_DEFINES)
 
 
@@ -493,28 +532,33 @@ def gemm_skinny_qkv_rope_supported(x: torch.Tensor, w: torch.Tensor, head_dim: i
 def gemm_skinny_qkv_rope(q_out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor,
                          block_table: torch.Tensor, block_size: int, cache: torch.Tensor, inv_freq: Optional[torch.Tensor],
                          rot_dim: int, is_neox: bool, n_q_heads: int, n_kv_heads: int, head_dim: int,
-                         error_flag: Optional[torch.Tensor] = None, prenorm=None):
+                         error_flag: Optional[torch.Tensor] = None, prenorm=None, bias: Optional[torch.Tensor] = None,
+                         kv_planes: int = 2, n_extra: int = 0):
     """The merged q, k, v projection of up to 16 single tokens (x [M, K] bfloat16, w [(heads + 2 kv heads) * head_dim, K])
     with the rotary encoding and the cache write in its epilogue: q_out [M, heads * head_dim] gets the rotated q, the
-    pages of `cache` the rotated k and v.  The same values as gemm_skinny followed by rope_cache_write.  prenorm: as in
-    `gemm_skinny`."""
+    pages of `cache` the rotated k and v.  The same values as gemm_skinny followed by rope_cache_write.  prenorm, bias: as in
+    `gemm_skinny`.  kv_planes 1: w has no v rows and the cache is [pages, 1, ...] (keys that are values).  n_extra: w has so
+    many rows behind them, whose results go to their own columns of q_out, [M, rows of w] then."""
     M, K = x.shape
     if (not gemm_skinny_qkv_rope_supported(x, w, head_dim, rot_dim if inv_freq is not None else 0, is_neox)
-            or w.shape != ((n_q_heads + 2 * n_kv_heads) * head_dim, K) or q_out.shape != (M, n_q_heads * head_dim)
+            or w.shape != ((n_q_heads + kv_planes * n_kv_heads) * head_dim + n_extra, K)
+            or q_out.shape != (M, w.shape[0] if n_extra else n_q_heads * head_dim) or kv_planes not in (1, 2)
             or q_out.dtype != torch.bfloat16 or q_out.stride(1) != 1):
         raise KernelError(f"gemm_skinny_qkv_rope: shapes {tuple(x.shape)} x {tuple(w.shape)}^T -> {tuple(q_out.shape)} are not taken")
-    if not cache.is_contiguous() or tuple(cache.shape[1:]) != (2, n_kv_heads, block_size, head_dim) or cache.dtype != torch.bfloat16:
+    _bf16_bias(bias, w.shape[0], "gemm_skinny_qkv_rope")
+    if not cache.is_contiguous() or tuple(cache.shape[1:]) != (kv_planes, n_kv_heads, block_size, head_dim) or cache.dtype != torch.bfloat16:
         raise KernelError(f"gemm_skinny_qkv_rope: cache of shape {tuple(cache.shape)} does not match the heads")
     if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dim // 2):
         raise KernelError("gemm_skinny_qkv_rope: inv_freq must be float32 [rot_dim / 2]")
     f = _func("gemm_skinny.cu", "lmsf_gemm_skinny_qkv_rope",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p,
                c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-               c_void_p, c_int, c_longlong, c_float, c_int, c_void_p], SKINNY_DEFINES)
+               c_void_p, c_int, c_longlong, c_float, c_int, c_void_p, c_int, c_int, c_void_p], SKINNY_DEFINES)
     rc = f(_ptr(q_out), q_out.stride(0), _ptr(x), x.stride(0), _ptr(w), w.stride(0), M, K, _i32(positions, "positions"),
            _i32(token_seq, "token_seq"), _i32(block_table, "block_table"), block_table.shape[1], block_size, _ptr(cache),
            cache.stride(0), _ptr(inv_freq) if inv_freq is not None else None, int(rot_dim), int(bool(is_neox)), n_q_heads,
-           n_kv_heads, head_dim, _i32(error_flag, "error_flag"), *_prenorm_args(prenorm, M, "gemm_skinny_qkv_rope"), _stream())
+           n_kv_heads, head_dim, _i32(error_flag, "error_flag"), *_prenorm_args(prenorm, M, "gemm_skinny_qkv_rope"),
+           _ptr(bias), int(kv_planes), int(n_extra), _stream())
     _check(rc, "gemm_skinny.cu", "lmsf_gemm_skinny", SKINNY_DEFINES)
 
 
@@ -626,13 +670,14 @@ def _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, wha
 
 
 
-def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=False, head_bias=None):
-    """(chunk, r1, r2, sinks, keep_first, sigmoid, head_bias) as the tensor-core attention kernels take them: what a design
+def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=False, head_bias=None, dist=None):
+    """(chunk, r1, r2, sinks, keep_first, sigmoid, head_bias, dist, its entries) as the tensor-core attention kernels take them: what a design
     adds to the causal softmax.  chunk > 0: a query at position p sees the keys p - p % chunk .. p only.  log_bias (r1, r2),
     float32 [n_q_heads] each: r1 * log(1 + r2 * distance) is taken off the scaled scores.  sinks, float32 [n_q_heads]:
     exp(sink) is one more term of the softmax's denominator.  keep_first (with a window): the request's first keys stay
     visible behind it.  sigmoid: a visible key's weight is sigmoid(score), not normalised.  head_bias, float32 [n_q_heads]:
-    added to the scaled scores."""
+    added to the scaled scores.  dist, float32 [n_q_heads, entries]: the entry of the distance (the last one for every larger
+    distance) is added to the scaled score."""
     _per_head(head_bias, n_q_heads, "the bias per head")
     r1, r2 = log_bias if log_bias is not None else (None, None)
     _per_head(r1, n_q_heads, "the logarithmic bias")
@@ -640,7 +685,8 @@ def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=
     _per_head(sinks, n_q_heads, "sinks")
     if chunk is not None and int(chunk) < 0:
         raise KernelError(f"attention: a chunk of {chunk} positions")
-    return int(chunk or 0), _ptr(r1), _ptr(r2), _ptr(sinks), int(keep_first or 0), 1 if sigmoid else 0, _ptr(head_bias)
+    return int(chunk or 0), _ptr(r1), _ptr(r2), _ptr(sinks), int(keep_first or 0), 1 if sigmoid else 0, _ptr(head_bias), \
+        *_dist_args(dist, n_q_heads)
 
 
 _DECODE_WIDTHS = {}
@@ -736,7 +782,7 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
                      ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int,
                      head_dim: int, n_splits: int, scratch: Optional[torch.Tensor], warps: int = 0, kv_planes: int = 2,
                      chunk: int = 0, log_bias=None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                     sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None):
+                     sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
     """Attention of requests that bring ONE query token each (row cu_q[s] of q), over their ctx_len[s] keys
     in pages.  seq_ids: int32 [n_served] rows of the block table that are served (None: all, in order).
     scratch: float32, at least attention_decode_scratch_floats(...) values when n_splits > 1, all zero when it is
@@ -745,7 +791,7 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
     kv_planes 1: the cache holds one vector per token and kv head that is key and value at once.
     chunk, log_bias, sinks: see _score_extras."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_decode", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
     n_total = block_table.shape[0]
     need = attention_decode_scratch_floats(n_total, n_q_heads, n_splits, head_dim)
     if need and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need):
@@ -756,7 +802,7 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
     f = _func("attention_mma.cu", "lmsf_attention_decode_width",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p,
-               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p], d)
+               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_ids, "seq_ids"), n_served, n_total,
            _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale), int(window or 0), n_q_heads, head_dim,
@@ -795,11 +841,11 @@ def attention_decode_items(out: torch.Tensor, q: torch.Tensor, cache: torch.Tens
                            scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int, warps: int,
                            scratch: torch.Tensor, kv_planes: int = 2, chunk: int = 0, log_bias=None,
                            sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                           sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None):
+                           sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
     """attention_decode with splits per request, over a list made by decode_build_items.  scratch: float32, at
     least attention_decode_items_scratch_floats(capacity, ...) values, zero when first used."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_decode_items", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
     need = attention_decode_items_scratch_floats(items.shape[0], n_q_heads, head_dim)
     if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
         raise KernelError(f"attention_decode_items: a list of {items.shape[0]} entries needs {need} float32 values of scratch")
@@ -807,7 +853,7 @@ def attention_decode_items(out: torch.Tensor, q: torch.Tensor, cache: torch.Tens
     f = _func("attention_mma.cu", "lmsf_attention_decode_items",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p, c_int,
-               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p], d)
+               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _ptr(items), items.shape[0], block_table.shape[0],
            _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale), int(window or 0), n_q_heads, head_dim, int(warps),
@@ -819,16 +865,16 @@ def attention_prefill(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, b
                       block_size: int, tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, cu_q: torch.Tensor,
                       ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int,
                       kv_planes: int = 2, chunk: int = 0, log_bias=None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                      sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None):
+                      sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
     """Attention of prompt portions.  Tile i covers the query tokens tile_q0[i] .. tile_q0[i] + 63 (counted
     inside the portion) of request tile_seq[i]."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_prefill", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
     d = _mma_defines(head_dim)
     f = _func("attention_mma.cu", "lmsf_attention_prefill",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int,
-               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p], d)
+               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _i32(tile_seq, "tile_seq"),
            _i32(tile_q0, "tile_q0"), n_tiles, _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale),
@@ -851,16 +897,16 @@ def attention_prefill_tc(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor
                          ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int,
                          error_flag: Optional[torch.Tensor] = None, kv_planes: int = 2, chunk: int = 0, log_bias=None,
                          sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                         sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None):
+                         sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
     """Attention of prompt portions on tcgen05 tensor cores (head size 64 or 128).  Tile i covers the query
     tokens tile_q0[i] .. tile_q0[i] + 127 (counted inside the portion) of request tile_seq[i]."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_prefill_tc", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
     d = _mma_defines(head_dim)[:1]
     f = _func("attention_tc.cu", "lmsf_attention_prefill_tc",
               [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_int, c_int,
                c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p,
-               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p], d)
+               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), cache.shape[0], block_size,
            n_kv_heads, _i32(block_table, "block_table"), block_table.shape[1], _i32(tile_seq, "tile_seq"),
            _i32(tile_q0, "tile_q0"), n_tiles, _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale),
@@ -926,6 +972,29 @@ def gated_branches(res: torch.Tensor, z: torch.Tensor, bias: Optional[torch.Tens
                c_void_p])
     rc = f(_ptr(res), _ptr(z), z.stride(0), _f32vec(bias, width, "bias"), _ptr(y1), _ptr(y2), _ptr(h),
            _f32vec(w_next, hidden, "w_next"), n, hidden, float(eps_next), dtype_code(y1.dtype), _stream())
+    _check(rc, "stream_norm.cu", "lmsf_stream_norm")
+
+
+def stream_branches(res: torch.Tensor, y1: Optional[torch.Tensor] = None, c1: float = 1.0, y2: Optional[torch.Tensor] = None,
+                    c2: float = 1.0, h1: Optional[torch.Tensor] = None, w1: Optional[torch.Tensor] = None,
+                    h2: Optional[torch.Tensor] = None, w2: Optional[torch.Tensor] = None, eps: float = 0.0):
+    """res += c1 * y1 + c2 * y2 (whichever is given), then h1 = norm(res) * w1 and h2 = norm(res) * w2 (whichever is given),
+    one root of the mean square for both; one kernel, float32 inside.  res: float32 [n, D]; y1, y2, h1, h2: contiguous [n, D]
+    of one activation type; w1, w2: float32 [D]."""
+    n, hidden = res.shape
+    if res.dtype != torch.float32 or not res.is_contiguous():
+        raise KernelError("stream_branches: the residual stream must be contiguous float32")
+    given = [t for t in (y1, y2, h1, h2) if t is not None]
+    if not given:
+        return
+    for t in given:
+        if t.shape != res.shape or not t.is_contiguous() or t.dtype != given[0].dtype:
+            raise KernelError("stream_branches: branches and outputs must be contiguous, of the stream's shape and of one type")
+    f = _func("stream_norm.cu", "lmsf_stream_branches",
+              [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
+               c_int, c_void_p])
+    rc = f(_ptr(res), _ptr(y1), float(c1), _ptr(y2), float(c2), _ptr(h1), _f32vec(w1, hidden, "w1"), _ptr(h2),
+           _f32vec(w2, hidden, "w2"), n, hidden, float(eps), dtype_code(given[0].dtype), _stream())
     _check(rc, "stream_norm.cu", "lmsf_stream_norm")
 
 
@@ -1125,10 +1194,11 @@ def gated_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
 
 
 def grouped_gated_norm(out: torch.Tensor, x: torch.Tensor, gate: Optional[torch.Tensor], w: torch.Tensor, group_size: int,
-                       eps: float, gate_act: str = "silu", gate_first: bool = False):
+                       eps: float, gate_act: str = "silu", gate_first: bool = False, out_scale: float = 1.0):
     """Per group of `group_size` columns: out = x / rms(x) * w * act(gate), or with gate_first out = y / rms(y) * w for
     y = x * act(gate).  x: float32 [n, width]; gate, out: [n, width] views of the activation type; w: float32, its length
-    divides into a row (a weight shorter than the row is shared by the groups)."""
+    divides into a row (a weight shorter than the row is shared by the groups).  out_scale multiplies the result before it
+    is rounded."""
     n, width = x.shape
     _rows(x, width, "grouped_gated_norm: x", torch.float32)
     _rows(out, width, "grouped_gated_norm: out")
@@ -1139,9 +1209,9 @@ def grouped_gated_norm(out: torch.Tensor, x: torch.Tensor, gate: Optional[torch.
         raise KernelError("grouped_gated_norm: the groups and the weight must divide a row")
     f = _func("recurrent.cu", "lmsf_grouped_gated_norm",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_float,
-               c_int, c_int, c_int, c_void_p])
+               c_int, c_int, c_float, c_int, c_void_p])
     rc = f(_ptr(out), out.stride(0), _ptr(x), x.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(w),
-           w.numel(), n, width // group_size, group_size, float(eps), int(gate_act == "silu"), int(gate_first),
+           w.numel(), n, width // group_size, group_size, float(eps), int(gate_act == "silu"), int(gate_first), float(out_scale),
            dtype_code(out.dtype), _stream())
     _check(rc, "recurrent.cu", "lmsf_recurrent")
 
@@ -1169,10 +1239,16 @@ def latent_norm_cache_write(x: torch.Tensor, w: torch.Tensor, eps: float, cache:
 
 def latent_norm_rope_cache_write(x: torch.Tensor, w: torch.Tensor, eps: float, cache: torch.Tensor, positions: torch.Tensor,
                                  token_seq: torch.Tensor, block_table: torch.Tensor, block_size: int, rank: int, rot_dim: int,
-                                 rot_n: int, inv_freq: Optional[torch.Tensor], error_flag: Optional[torch.Tensor] = None):
+                                 rot_n: int, inv_freq: Optional[torch.Tensor], error_flag: Optional[torch.Tensor] = None,
+                                 interleaved: bool = False, rot_mult: float = 1.0, q_rank: int = 0,
+                                 wq: Optional[torch.Tensor] = None, q_out: Optional[torch.Tensor] = None,
+                                 write: bool = True):
     """cache[page of token t][slot] = [norm(x[t, :rank]) * w | key part | zeros]: the key part x[t, rank:rank + rot_dim] has
     its first rot_n values rotated by the token's position (value i pairs with value i + rot_n / 2; inv_freq float32
-    [rot_n / 2]).  x: [n, rank + rot_dim] view; cache: [pages, 1, 1, block_size, padded]."""
+    [rot_n / 2]).  x: [n, rank + rot_dim] view; cache: [pages, 1, 1, block_size, padded].  interleaved: value 2 i pairs with
+    value 2 i + 1; rot_mult multiplies cos and sin.  q_rank > 0: the q_rank values before x in the same rows (x is a view
+    into them) are normed with wq (float32 [q_rank]) into q_out ([n, q_rank]) by the same launch.  write False: nothing is
+    cached."""
     n = x.shape[0]
     padded = cache.shape[-1]
     if x.shape != (n, rank + rot_dim) or x.stride(1) != 1 or cache.dtype != x.dtype or not cache.is_contiguous() or \
@@ -1180,20 +1256,25 @@ def latent_norm_rope_cache_write(x: torch.Tensor, w: torch.Tensor, eps: float, c
         raise KernelError(f"latent cache: x [n, {rank + rot_dim}] and a cache [pages, 1, 1, {block_size}, >= {rank + rot_dim}] of one dtype")
     if rot_n and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_n // 2 or not inv_freq.is_contiguous()):
         raise KernelError("latent cache: inv_freq must hold rot_n / 2 float32 values")
+    if q_rank and (q_out is None or wq is None or q_out.shape != (n, q_rank) or not q_out.is_contiguous() or q_out.dtype != x.dtype
+                   or x.storage_offset() < q_rank or x.stride(0) < q_rank + rank + rot_dim):
+        raise KernelError(f"latent cache: q_out must be contiguous [n, {q_rank}] and x a view behind {q_rank} values of its rows")
     f = _func("latent_cache.cu", "lmsf_latent_norm_rope_cache_write",
               [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-               c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p])
-    rc = f(_ptr(x), x.stride(0), _f32vec(w, rank, "w"), _ptr(cache), cache.stride(0), _i32(positions, "positions"),
+               c_int, c_float, c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+    rc = f(_ptr(x), x.stride(0), _f32vec(w, rank, "w"), _ptr(cache) if write else None, cache.stride(0), _i32(positions, "positions"),
            _i32(token_seq, "token_seq"), _i32(block_table, "block_table"), block_table.shape[1], block_size, n, rank, padded,
-           float(eps), int(rot_dim), int(rot_n), _ptr(inv_freq), dtype_code(x.dtype), _i32(error_flag, "error_flag"), _stream())
+           float(eps), int(rot_dim), int(rot_n), _ptr(inv_freq), int(bool(interleaved)), float(rot_mult), int(q_rank),
+           _f32vec(wq, q_rank, "wq") if q_rank else None, _ptr(q_out) if q_rank else None, dtype_code(x.dtype), _i32(error_flag, "error_flag"), _stream())
     _check(rc, "latent_cache.cu", "lmsf_latent_cache")
 
 
 def latent_query_rope(qa: torch.Tensor, q: torch.Tensor, positions: torch.Tensor, heads: int, plain: int, rot_dim: int,
-                      rot_n: int, inv_freq: Optional[torch.Tensor], rank: int, padded: int):
+                      rot_n: int, inv_freq: Optional[torch.Tensor], rank: int, padded: int, interleaved: bool = False,
+                      rot_mult: float = 1.0):
     """qa[t, h, rank:rank + rot_dim] = the rotated part q[t, h, plain:plain + rot_dim] of every head, its first rot_n values
     rotated by the token's position; qa[t, h, rank + rot_dim:padded] = 0.  q: [n, heads * (plain + rot_dim)] view,
-    qa: [n, heads * padded]."""
+    qa: [n, heads * padded].  interleaved, rot_mult: as in latent_norm_rope_cache_write."""
     n = q.shape[0]
     if q.shape != (n, heads * (plain + rot_dim)) or q.stride(1) != 1 or qa.shape != (n, heads * padded) or qa.stride(1) != 1 \
             or qa.dtype != q.dtype:
@@ -1201,10 +1282,10 @@ def latent_query_rope(qa: torch.Tensor, q: torch.Tensor, positions: torch.Tensor
     if rot_n and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_n // 2 or not inv_freq.is_contiguous()):
         raise KernelError("latent query: inv_freq must hold rot_n / 2 float32 values")
     f = _func("latent_cache.cu", "lmsf_latent_query_rope",
-              [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
-               c_int, c_void_p])
+              [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float,
+               c_int, c_int, c_int, c_void_p])
     rc = f(_ptr(q), q.stride(0), _ptr(qa), qa.stride(0), _i32(positions, "positions"), n, heads, plain, rot_dim, int(rot_n),
-           _ptr(inv_freq), rank, padded, dtype_code(q.dtype), _stream())
+           _ptr(inv_freq), int(bool(interleaved)), float(rot_mult), rank, padded, dtype_code(q.dtype), _stream())
     _check(rc, "latent_cache.cu", "lmsf_latent_cache")
 
 
@@ -1437,3 +1518,98 @@ def relu2_(x: torch.Tensor):
     f = _func("moe.cu", "lmsf_relu2", [c_void_p, c_longlong, c_int, c_void_p])
     rc = f(_ptr(x), x.numel(), dtype_code(x.dtype), _stream())
     _check(rc, "moe.cu", "lmsf_moe")
+
+
+# ----------------------------------------------------------------------------- a matrix memory with exponential gates
+
+MEMORY_MAX_DK = 256
+_MEMORY_CHUNK: Optional[int] = None
+
+
+def matrix_memory_chunk_tokens() -> int:
+    """Most tokens of a chunk of a long portion (a constant of csrc/matrix_memory.cu)."""
+    global _MEMORY_CHUNK
+    if _MEMORY_CHUNK is None:
+        lib = load_library("matrix_memory.cu")
+        lib.lmsf_matrix_memory_chunk_tokens.restype = c_int
+        _MEMORY_CHUNK = int(lib.lmsf_matrix_memory_chunk_tokens())
+    return _MEMORY_CHUNK
+
+
+MEMORY_COLS = 64      # value columns per block: every such tile of a slot's state has copies of n and m of its own
+
+
+def matrix_memory_state_floats(heads: int, dk: int, dv: int) -> int:
+    """Floats of a state slot: S [heads, dk, dv], then per tile of 64 value columns n [heads, dk], then per tile m [heads]."""
+    tiles = -(-dv // MEMORY_COLS)
+    return heads * dk * (dv + tiles) + tiles * heads
+
+
+def matrix_memory(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gi: torch.Tensor, gf: torch.Tensor,
+                  bi: torch.Tensor, bf: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, state_slot: torch.Tensor,
+                  n_seqs: int, heads: int, dk: int, dv: int, cap: float, q_scale: float, eps: float = 1e-6,
+                  items: Optional[torch.Tensor] = None, spans: Optional[torch.Tensor] = None,
+                  last_chunk: Optional[torch.Tensor] = None):
+    """Per request (tokens cu_q[s]..cu_q[s + 1]) and head, with log gates i = cap tanh((gi + bi) / cap) and f = log sigmoid(cap
+    tanh((gf + bf) / cap)): m' = max(f + m, i), S = exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone, out = S^T q /
+    (max(|n . q|, exp(-m')) + eps), q times q_scale.  state: float32 [slots, matrix_memory_state_floats(...)], read before and
+    written after.  q, k: [n, heads * dk], v: [n, heads * dv], gi, gf: [n, heads]: views of one type; out: float32 [n, heads * dv].
+    items (int32 [*, 4]: request, first token, end token, chunk index): the launch serves these instead of every request whole;
+    with spans (int32 [*, 4]: request, first item, end item, 0) they are chunks of at most matrix_memory_chunk_tokens() tokens
+    of long portions (three launches), and last_chunk (int32 per item) marks each portion's last."""
+    n = q.shape[0]
+    for name, t, width in (("q", q, heads * dk), ("k", k, heads * dk), ("v", v, heads * dv), ("gi", gi, heads), ("gf", gf, heads)):
+        if t.shape[0] != n:
+            raise KernelError(f"matrix_memory: {name} must have {n} rows")
+        _rows(t, width, f"matrix_memory: {name}", q.dtype)
+    _rows(out, heads * dv, "matrix_memory: out", torch.float32)
+    if gi.stride(0) != gf.stride(0):
+        raise KernelError("matrix_memory: the two gates' logits must share one row stride")
+    if state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or \
+            state.shape[1] < matrix_memory_state_floats(heads, dk, dv):
+        raise KernelError("matrix_memory: the state must be contiguous float32 [slots, matrix_memory_state_floats(...)]")
+    for name, t in (("items", items), ("spans", spans)):
+        if t is not None and (t.dtype != torch.int32 or t.dim() != 2 or t.shape[1] != 4 or not t.is_contiguous()):
+            raise KernelError(f"matrix_memory: {name} must be a contiguous int32 tensor [n, 4]")
+    n_items = items.shape[0] if items is not None else n_seqs
+    scratch = None
+    if spans is not None:
+        if items is None or last_chunk is None or last_chunk.numel() != n_items:
+            raise KernelError("matrix_memory: chunks need their list and one mark per item")
+        need = _func("matrix_memory.cu", "lmsf_matrix_memory_scratch_floats", [c_int, c_int, c_int, c_int])
+        need.restype = c_longlong
+        scratch = torch.empty(int(need(n_items, heads, dk, dv)), dtype=torch.float32, device=q.device)
+    f = _func("matrix_memory.cu", "lmsf_matrix_memory",
+              [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
+               c_float, c_float, c_float, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int,
+               c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p])
+    rc = f(_ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), _ptr(gi), _ptr(gf), gi.stride(0),
+           _f32vec(bi, heads, "bi"), _f32vec(bf, heads, "bf"), float(cap), float(q_scale), float(eps), _ptr(out), out.stride(0),
+           _ptr(state), state.stride(0), _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), n_items, heads, dk, dv,
+           dtype_code(q.dtype), _ptr(items), _ptr(spans), spans.shape[0] if spans is not None else 0, _i32(last_chunk, "last_chunk"),
+           _ptr(scratch), _stream())
+    _check(rc, "matrix_memory.cu", "lmsf_matrix_memory")
+    if spans is not None:
+        add_launches(2)
+
+
+# ----------------------------------------------------------------------------- a gated recurrence element by element
+
+def min_gru(out: torch.Tensor, z: torch.Tensor, u: torch.Tensor, g: torch.Tensor, bz: Optional[torch.Tensor],
+            bu: Optional[torch.Tensor], state: torch.Tensor, cu_q: torch.Tensor, state_slot: torch.Tensor, n_seqs: int, max_q: int):
+    """Per request and channel: z' = sigmoid(z + bz), u' = u + bu, candidate c = u' + 1/2 where u' >= 0, sigmoid(u') elsewhere;
+    S = (1 - z') S + z' c; out = S * silu(g).  z, u, g: [n, width] views of one type and row stride; out: [n, width] of that
+    type; bz, bu: float32 [width]; state: float32 [slots, width], read before and written after.  max_q: the longest portion."""
+    n, width = z.shape
+    for name, t in (("z", z), ("u", u), ("g", g), ("out", out)):
+        _rows(t, width, f"min_gru: {name}", z.dtype)
+        if t.shape[0] != n or (name != "out" and t.stride(0) != z.stride(0)):
+            raise KernelError("min_gru: z, u, g and out have one number of rows, z, u and g one row stride")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] != width or not state.is_contiguous():
+        raise KernelError(f"min_gru: the state must be contiguous float32 [slots, {width}]")
+    f = _func("min_gru.cu", "lmsf_min_gru",
+              [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
+               c_int, c_int, c_int, c_int, c_void_p])
+    rc = f(_ptr(z), _ptr(u), _ptr(g), z.stride(0), _f32vec(bz, width, "bz"), _f32vec(bu, width, "bu"), _ptr(out), out.stride(0),
+           _ptr(state), _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), n_seqs, int(max_q), width, dtype_code(z.dtype), _stream())
+    _check(rc, "min_gru.cu", "lmsf_min_gru")

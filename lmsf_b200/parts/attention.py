@@ -41,14 +41,15 @@ class PagedAttention(Mixer):
                  qk_norm_weights: bool = True, value_norm: bool = False, chunk: Optional[int] = None,
                  head_gate: bool = False, keep_first: int = 0, score_weights: str = "softmax", head_bias: bool = False,
                  value_gate: bool = False, own_kv: bool = True, cache_window="own",
-                 cache_keep_first: Optional[int] = None):
+                 cache_keep_first: Optional[int] = None, values_are_keys: bool = False, unit_sink: bool = False,
+                 out_bias: Optional[bool] = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot be grouped over {num_kv_heads} kv heads")
         # head_dim is the stored size of a query or key head, value_dim that of a value head (default: the same).  The
         # cache and the kernels work on ONE width per head, a multiple of 16; where the stored sizes differ from it the
         # weights are padded with zero rows and columns when they are set (zeros change neither scores nor outputs)
         self.qk_dim, self.value_dim = int(head_dim), int(value_dim or head_dim)
-        padded = value_dim is not None or qk_norm
+        padded = value_dim is not None or qk_norm or values_are_keys
         width = (max(self.qk_dim, self.value_dim) + 15) // 16 * 16 if padded else head_dim
         if width % 16 or not (16 <= width <= 256):
             raise ValueError(f"head_dim {head_dim} is not supported: the attention kernels take multiples of 16 "
@@ -90,6 +91,15 @@ class PagedAttention(Mixer):
         # ("own": what this part's mask needs; None: every key; a number: a window of that size)
         self.cache_window = (int(window) if window else None) if cache_window == "own" else (int(cache_window) if cache_window else None)
         self.cache_keep_first = int(cache_keep_first) if cache_keep_first is not None else self.keep_first
+        # values_are_keys: a token's value is its key (as it stands in the cache); there is no value projection and the cache
+        # holds one vector per token and kv head.  unit_sink: one is added to the softmax's denominator (a sink of score 0)
+        self.values_are_keys, self.unit_sink = bool(values_are_keys), bool(unit_sink)
+        self.kv_planes = 1 if self.values_are_keys else 2
+        if self.values_are_keys and (self.value_dim != self.qk_dim or qk_norm or self.head_gate or self.value_gate or not self.own_kv):
+            raise ValueError("values that are the keys have the keys' size and are not built with norms, gates or another call's keys")
+        if self.unit_sink and self.sigmoid_weights:
+            raise ValueError("a sink belongs to a softmax, not to sigmoid weights")
+        self._sinks: Optional[torch.Tensor] = None
         self.head_bias: Optional[torch.Tensor] = None
         self._hb32: Optional[torch.Tensor] = None
         self.q_norm: Optional[torch.Tensor] = None
@@ -105,6 +115,7 @@ class PagedAttention(Mixer):
         self.q_size = num_heads * head_dim
         self.kv_size = num_kv_heads * head_dim
         self.has_bias = bool(bias)
+        self.has_out_bias = self.has_bias if out_bias is None else bool(out_bias)
         self.qkv: Optional[torch.Tensor] = None
         self.o: Optional[torch.Tensor] = None
         self.qkv_bias: Optional[torch.Tensor] = None
@@ -112,13 +123,14 @@ class PagedAttention(Mixer):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         H, G, dk, dv, D = self.num_heads, self.num_kv_heads, self.qk_dim, self.value_dim, self.hidden_size
-        merged = [(H * dk, D)] + ([(G * dk, D), (G * dv, D)] if self.own_kv else [])
+        merged = [(H * dk, D)] + ([(G * dk, D)] if self.values_are_keys else [(G * dk, D), (G * dv, D)] if self.own_kv else [])
         merged += ([(H, D)] if self.head_gate else []) + ([(H * dv, D)] if self.value_gate else [])
         specs = {"qkv": WeightSpec(merged), "o": WeightSpec([(D, H * dv)])}
         if self.has_head_bias:
             specs["head_bias"] = WeightSpec([(H,)], keep_fp32=True)
         if self.has_bias:
-            specs["qkv_bias"] = WeightSpec([(H * dk,), (G * dk,), (G * dv,)])
+            specs["qkv_bias"] = WeightSpec([(H * dk,), (G * dk,)] + ([] if self.values_are_keys else [(G * dv,)]))
+        if self.has_out_bias:
             specs["o_bias"] = WeightSpec([(D,)])
         if self.qk_norm and self.qk_norm_weights:
             specs["q_norm"] = WeightSpec([(dk,)], keep_fp32=True)
@@ -137,7 +149,10 @@ class PagedAttention(Mixer):
                 return out.reshape(heads * hd, *t.shape[2:])
 
             for name in ("qkv", "qkv_bias"):
-                if name in tensors and not self.own_kv:
+                if name in tensors and self.values_are_keys:
+                    t = tensors[name]
+                    tensors[name] = torch.cat([pad_heads(t[:H * dk], H, dk), pad_heads(t[H * dk:], G, dk)], 0).contiguous()
+                elif name in tensors and not self.own_kv:
                     t = tensors[name]
                     tensors[name] = torch.cat([pad_heads(t[:H * dk], H, dk), t[H * dk:]], 0).contiguous()
                 elif name in tensors:
@@ -159,7 +174,7 @@ class PagedAttention(Mixer):
         super().set_weights(tensors)
 
     def cache_spec(self) -> Optional[KVCacheSpec]:
-        return KVCacheSpec(self.num_kv_heads, self.head_dim, self.cache_window,
+        return KVCacheSpec(self.num_kv_heads, self.head_dim, self.cache_window, planes=self.kv_planes,
                            keep_first=self.cache_keep_first if self.cache_window else 0)
 
     def activation_width(self) -> int:
@@ -171,6 +186,8 @@ class PagedAttention(Mixer):
             self.position_encoding.prepare(dtype, device)
         if self.qk_norm and self.qk_norm_weights:
             self._qn32, self._kn32 = self.q_norm.float().contiguous(), self.k_norm.float().contiguous()
+        if self.unit_sink:
+            self._sinks = torch.zeros(self.num_heads, dtype=torch.float32, device=device)
         if self.has_head_bias:
             self._hb32 = self.head_bias.float().contiguous()
         if dtype == torch.bfloat16 and not kernels.mma_attention_supported(dtype, self.head_dim):
@@ -192,7 +209,53 @@ class PagedAttention(Mixer):
         f = getattr(self.position_encoding, "score_log_bias", None)
         return f() if f is not None else None
 
+    def _dist_table(self) -> Optional[torch.Tensor]:
+        return self.position_encoding.score_distance_table() if self.position_encoding is not None else None
+
+    def project(self, ctx: StepContext, h, w: torch.Tensor, bias: Optional[torch.Tensor], cache: LayerCache):
+        """h times a matrix whose first rows are this part's merged one (values that are the keys only): (product, whether its
+        keys are in the cache already).  A few single tokens: the product's epilogue writes the keys to their pages (their
+        columns of the product are then not set)."""
+        hx = h.x if isinstance(h, Prenormed) else h
+        n_extra = w.shape[0] - self.q_size - self.kv_size
+        if (FUSE_QKV_ROPE and cache.owner and linear.USE_SKINNY and self._no_rotation()
+                and kernels.gemm_skinny_qkv_rope_supported(hx, w, self.head_dim, 0, True)):
+            group = ctx.groups[cache.group]
+            p = torch.empty((ctx.n_tokens, w.shape[0] if n_extra else self.q_size), dtype=hx.dtype, device=hx.device)
+            kernels.gemm_skinny_qkv_rope(p, hx, w, ctx.positions, ctx.token_seq, group.block_table, group.block_size, cache.kv,
+                                         None, 0, True, self.num_heads, self.num_kv_heads, self.head_dim, ctx.error_flag,
+                                         prenorm=(h.sumsq, h.eps, h.width) if isinstance(h, Prenormed) else None, bias=bias,
+                                         kv_planes=1, n_extra=n_extra)
+            return p, True
+        return matmul_tn(h, w, bias=bias), False
+
+    def _no_rotation(self) -> bool:
+        """Whether q and k pass as they are projected (positions, if any, enter the scores)."""
+        return self.position_encoding is None or self._dist_table() is not None or self._slopes() is not None or \
+            self._log_bias() is not None
+
+    def attend_projected(self, ctx: StepContext, p: torch.Tensor, cached: bool, cache: LayerCache, out: torch.Tensor) -> None:
+        """What follows `project`: keys into their pages (unless they are there), positions, attention; the heads' outputs go
+        to `out` [n, q_size] (a view whose rows are 16-byte aligned)."""
+        group = ctx.groups[cache.group]
+        fused = self.position_encoding.fused_rotary() if self.position_encoding is not None else None
+        if fused is None and not self._no_rotation():
+            raise ValueError("values that are the keys take a rotary encoding, a bias on the scores or none")
+        inv_freq, rot_dim, is_neox = fused if fused is not None else (None, 0, True)
+        q = p[:, :self.q_size]
+        if not cached and (cache.owner or fused is not None):
+            k = p[:, self.q_size:self.q_size + self.kv_size]
+            kernels.rope_cache_write(q, k, None, ctx.positions, ctx.token_seq, group.block_table, group.block_size,
+                                     cache.kv if cache.owner else None, inv_freq, rot_dim, is_neox, self.num_heads,
+                                     self.num_kv_heads, self.head_dim, ctx.error_flag)
+        self.attend(ctx, out, q, cache.kv, group)
+
     def forward(self, ctx: StepContext, h, cache: LayerCache, then: Optional[NormAfter] = None):
+        if self.values_are_keys:
+            p, cached = self.project(ctx, h, self.qkv, self.qkv_bias, cache)
+            out = torch.empty((ctx.n_tokens, self.q_size), dtype=p.dtype, device=p.device)
+            self.attend_projected(ctx, p, cached, cache, out)
+            return self._project_out(out, then)
         group = ctx.groups[cache.group]
         fused = self.position_encoding.fused_rotary() if self.position_encoding is not None else None
         hx = h.x if isinstance(h, Prenormed) else h
@@ -238,7 +301,7 @@ class PagedAttention(Mixer):
             k = v = None
             if self.head_gate:
                 gate = matmul_tn(h, self.qkv[self.q_size + 2 * self.kv_size:])[:, :self.num_heads]
-        if self.position_encoding is not None and fused is None and self._slopes() is None and self._log_bias() is None:
+        if self.position_encoding is not None and fused is None and not self._no_rotation():
             if self.qk_norm:
                 raise ValueError("a norm of queries and keys goes with a rotary encoding, a bias on the scores or none")
             self.position_encoding.apply(ctx, q, k, self.num_heads, self.num_kv_heads, self.head_dim)
@@ -271,28 +334,28 @@ class PagedAttention(Mixer):
         paged_attend(ctx, out, q, kv, group, num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
                      scale=self.scale, window=self.window, softcap=self.softcap, slopes=self._slopes(), chunk=self.chunk,
                      log_bias=self._log_bias(), gate=gate, keep_first=self.keep_first, sigmoid=self.sigmoid_weights,
-                     head_bias=self._hb32)
+                     head_bias=self._hb32, sinks=self._sinks, dist=self._dist_table(), kv_planes=self.kv_planes)
 
 
 def paged_attend(ctx: StepContext, out: torch.Tensor, q: torch.Tensor, kv: torch.Tensor, group, *, num_heads: int,
                  num_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None, softcap: float = 0.0,
                  slopes: Optional[torch.Tensor] = None, kv_planes: int = 2, chunk: Optional[int] = None,
                  log_bias=None, gate: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                 keep_first: int = 0, sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None) -> None:
+                 keep_first: int = 0, sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None,
+                 dist: Optional[torch.Tensor] = None) -> None:
     """Attention over pages for any mix of tokens.  bfloat16 with a head size up to 256: single tokens go to the
     split-key decode kernel, longer portions to a tiled prefill kernel (tcgen05 with accumulators in tensor memory for
     head sizes 64 and 128, mma.sync otherwise).  Everything else, float32 included, runs on the generic kernel, which is
-    also their plain twin.  kv_planes 1: one cached vector per token and kv head is key and value at once (the fast
-    kernels only; the caller keeps its own plain kernel for that layout).  chunk: a query sees the keys of its own chunk of
+    also their plain twin.  kv_planes 1: one cached vector per token and kv head is key and value at once.  chunk: a query sees the keys of its own chunk of
     positions only; log_bias (r1, r2): r1 * log(1 + r2 * distance) is taken off the scores; sinks [heads]: exp(sink) joins
     the softmax's denominator (all three: every kernel); gate [n, heads]: the output of head h is multiplied by
     sigmoid(gate[:, h]) (the generic kernel itself, a small kernel after the fast ones).  keep_first: with a window, the
     request's first keys stay visible behind it; sigmoid: a key's weight is sigmoid(score), not normalised; head_bias [heads]:
-    added to the scaled scores."""
+    added to the scaled scores; dist [heads, entries]: a number per (head, distance) added to them."""
     if kernels.mma_attention_supported(q.dtype, head_dim) and not softcap and slopes is None and \
             not ctx.extras.get("force_generic_attention"):
         extras = dict(chunk=chunk or 0, log_bias=log_bias, sinks=sinks, keep_first=keep_first if window else 0,
-                      sigmoid=sigmoid, head_bias=head_bias)
+                      sigmoid=sigmoid, head_bias=head_bias, dist=dist)
         if ctx.n_decode_seqs:
             max_ctx = ctx.extras.get("decode_max_ctx")
             if max_ctx is None:
@@ -362,9 +425,8 @@ def paged_attend(ctx: StepContext, out: torch.Tensor, q: torch.Tensor, kv: torch
         if gate is not None:
             kernels.head_gate_(out, gate, num_heads, head_dim)
         return
-    if kv_planes != 2:
-        raise ValueError("the plain attention kernel of keys and values takes a cache of two planes")
     kernels.attention_generic(out, q, kv, group.block_table, group.block_size, ctx.token_seq, ctx.positions,
                               scale, window or 0, num_heads, num_kv_heads, head_dim,
                               softcap=softcap, slopes=slopes, chunk=chunk or 0, log_bias=log_bias, gate=gate, sinks=sinks,
-                              keep_first=keep_first if window else 0, sigmoid=sigmoid, head_bias=head_bias)
+                              keep_first=keep_first if window else 0, sigmoid=sigmoid, head_bias=head_bias, dist=dist,
+                              kv_planes=kv_planes)

@@ -65,12 +65,26 @@ class ModelSpec:
     entries: List[PartSpec] = field(default_factory=list)        # family "stream_entry", named by LayerCall.entry
 
 
+ANY_SIZE = -1      # in a WeightSpec's shape: a size that the stored tensor gives
+
+
 @dataclass
 class WeightSpec:
-    """Shapes of the source tensors (concatenated along dim 0, in order).  `keep_fp32`: a source
+    """Shapes of the source tensors (concatenated along dim 0, in order); ANY_SIZE stands for a size that the stored tensor
+    gives (`free_size` where there is no file: random weights).  `keep_fp32`: a source
     stored in 32-bit stays float32 even when the run dtype is bfloat16 (norm weights, biases)."""
     shapes: List[Tuple[int, ...]]
     keep_fp32: bool = False
+    free_size: int = 16
+
+    def matches(self, i: int, shape) -> bool:
+        """Whether a stored tensor's shape is that of source i."""
+        want = self.shapes[i]
+        return len(want) == len(shape) and all(w in (ANY_SIZE, s) for w, s in zip(want, shape))
+
+    def concrete(self, i: int) -> Tuple[int, ...]:
+        """Source i's shape with the free sizes filled in."""
+        return tuple(self.free_size if w == ANY_SIZE else w for w in self.shapes[i])
 
 
 @dataclass(frozen=True)
@@ -261,6 +275,11 @@ class PositionEncoding(Part):
         slope * (key position - query position); None otherwise."""
         return None
 
+    def score_distance_table(self) -> Optional[torch.Tensor]:
+        """float32 [query heads, entries] when the encoding adds a number per (head, distance) to the scaled scores, the last
+        entry serving every larger distance; None otherwise."""
+        return None
+
 
 class Shift(Part):
     """Mixes every token's row with the row of the token before it in the same request, which is the request's state between
@@ -278,6 +297,8 @@ class Mixer(Part):
     # may return a `Prenormed`.  A part that says neither is always given and asked for plain tensors.
     takes_prenormed = False
     fuses_norm = False
+    # what the block multiplies the output by where it adds it to the stream; only blocks that say `scales_mixer` do
+    out_scale = 1.0
 
     def cache_spec(self) -> Optional[KVCacheSpec]:
         return None
@@ -327,6 +348,7 @@ class Block:
         return None
 
     fuses_next_norm = False
+    scales_mixer = False        # the block multiplies its mixer's output by `Mixer.out_scale`
 
 
 # ----------------------------------------------------------------------------- registries
@@ -357,11 +379,12 @@ def part_class(family: str, kind: str):
 def build_part(family: str, spec: PartSpec) -> Part:
     params = dict(spec.params)
     # a nested PartSpec is built first; its key names its family
-    # (e.g. params["position_encoding"] of an attention mixer)
+    # (e.g. params["position_encoding"] of an attention mixer; "mixer_left" and "mixer_right" are two of one family)
     nested = []
     for k, v in list(params.items()):
         if isinstance(v, PartSpec):
-            params[k] = build_part(k, v)
+            fam = k if k in _REGISTRY else next((f for f in FAMILIES if k.startswith(f + "_")), k)
+            params[k] = build_part(fam, v)
             nested.append((params[k], v))
     part = part_class(family, spec.kind)(**params)
     part.nested_parts = nested        # parts with weights of their own are loaded like any other

@@ -225,3 +225,78 @@ class ParallelGatedBlock(Block):
                                w_next=nxt.weight_f32() if nxt is not None else None,
                                eps_next=nxt.eps if nxt is not None else 0.0)
         return (Normed(h_next, nxt, res) if nxt is not None else None), res
+
+
+@register_part("block", "parallel_norms")
+class ParallelNormsBlock(Block):
+    """Two branches side by side, each behind a norm of its own over the same stream:
+         x <- x + (mixer(norm1(x)) + ff(norm2(x)))
+    The norms share the root of the mean square, so one kernel ends a layer: both branches' sum into the float32 stream and,
+    when the next block is of this kind, both of its norms (`kernels.stream_branches`).  The mixer's output is multiplied by
+    its `out_scale` there, in float32.  A layer may have no feed-forward (and then no second norm)."""
+    ROLES = {"mixer_norm": "norm", "mixer": "mixer", "ffn_norm": "norm", "feed_forward": "feed_forward"}
+    OPTIONAL_ROLES = ("ffn_norm", "feed_forward")
+    fuses_next_norm = True
+    scales_mixer = True
+
+    def __init__(self, parts: Dict[str, Part]):
+        super().__init__(parts)
+        self.mixer_norm, self._mixer = parts["mixer_norm"], parts["mixer"]
+        self.ffn_norm, self.feed_forward = parts.get("ffn_norm"), parts.get("feed_forward")
+        if (self.feed_forward is None) != (self.ffn_norm is None):
+            raise ValueError("a feed-forward and its norm go together")
+        for n in (self.mixer_norm, self.ffn_norm):
+            if n is not None and (not hasattr(n, "weight_f32") or getattr(n, "has_layer_scale", False)):
+                raise ValueError("the block takes norms that are a factor per row times a weight (rmsnorm)")
+        if self.ffn_norm is not None and self.ffn_norm.eps != self.mixer_norm.eps:
+            raise ValueError("the block's two norms share one eps")
+
+    def entry(self) -> Optional[Tuple[Norm, Part]]:
+        return ParallelNorms(self.mixer_norm, self.ffn_norm), self._mixer
+
+    @staticmethod
+    def _end(ctx: StepContext, res: torch.Tensor, a, c: float, f, norms: Optional["ParallelNorms"]):
+        """res += c * a + f; the two normed forms of it that `norms` asks for."""
+        h1 = h2 = None
+        if norms is not None:
+            h1 = torch.empty(res.shape, dtype=ctx.dtype, device=res.device)
+            h2 = torch.empty_like(h1) if norms.second is not None else None
+        kernels.stream_branches(res, a, c, f, 1.0, h1, norms.first.weight_f32() if norms is not None else None, h2,
+                                norms.second.weight_f32() if h2 is not None else None,
+                                norms.first.eps if norms is not None else 0.0)
+        return h1, h2
+
+    def forward(self, ctx: StepContext, x, res: Optional[torch.Tensor], cache: LayerCache,
+                next_entry: Optional[Tuple[Norm, Part]] = None):
+        if isinstance(x, Normed):
+            if not isinstance(x.norm, ParallelNorms) or x.norm.first is not self.mixer_norm or x.res is not res:
+                raise ValueError("a prepared activation was made for other norms or another residual stream")
+            h1, h2 = x.h
+        else:
+            if x is not None and res is None:       # the embedding's output starts the stream
+                res = x if x.dtype == torch.float32 else torch.empty(x.shape, dtype=torch.float32, device=x.device)
+                if res is not x:
+                    kernels.stream_begin(res, x)
+                x = None
+            h1, h2 = self._end(ctx, res, x, 1.0, None, ParallelNorms(self.mixer_norm, self.ffn_norm))
+        a = self._mixer.forward(ctx, h1, cache)
+        f = self.feed_forward.forward(ctx, h2) if self.feed_forward is not None else None
+        norms = None
+        if next_entry is not None:
+            n = next_entry[0]
+            if isinstance(n, ParallelNorms):
+                norms = n
+            elif hasattr(n, "weight_f32") and not getattr(n, "has_layer_scale", False):
+                norms = ParallelNorms(n, None)
+        h1, h2 = self._end(ctx, res, a, self._mixer.out_scale, f, norms)
+        if norms is None:
+            return None, res
+        return (Normed((h1, h2), norms, res) if isinstance(next_entry[0], ParallelNorms) else Normed(h1, norms.first, res)), res
+
+
+class ParallelNorms:
+    """The two norms that a parallel-norms block applies to the stream (the second may be missing); what stands for its first
+    norm when the block before is asked to apply it."""
+
+    def __init__(self, first: Norm, second: Optional[Norm]):
+        self.first, self.second = first, second

@@ -35,6 +35,9 @@ class DecoderModel:
                 parts[role] = build_part(family, ls.parts[role])
                 self._owned += list(with_nested(parts[role], ls.parts[role]))
             self.blocks.append(cls(parts, **ls.block_params))
+            m = self.blocks[-1].mixer
+            if m is not None and m.out_scale != 1.0 and not cls.scales_mixer:
+                raise ValueError(f"block {ls.block!r} does not multiply its mixer's output, which asks for a factor {m.out_scale}")
         self.final_norm = build_part("norm", spec.final_norm)
         self.lm_head = build_part("linear", spec.lm_head)
         self._owned += [*with_nested(self.final_norm, spec.final_norm), *with_nested(self.lm_head, spec.lm_head)]

@@ -30,18 +30,10 @@ class TokenEmbedding(Part):
         return x
 
     def forward_stream(self, ctx: StepContext, keep: bool = False):
-        """(stream, copy of it or None), both float32 [n_tokens, hidden]."""
-        x = self.forward(ctx)
-        if x.dtype == torch.float32:
-            res = x
-        else:
-            res = torch.empty(x.shape, dtype=torch.float32, device=x.device)
-            kernels.stream_begin(res, x)
-        first = None
-        if keep:
-            first = torch.empty_like(res)
-            kernels.stream_begin(first, x)
-        return res, first
+        """(stream, copy of it or None), both float32 [n_tokens, hidden]; the scaled row is not rounded on the way."""
+        res = torch.empty((ctx.n_tokens, self.hidden_size), dtype=torch.float32, device=self.weight.device)
+        kernels.embedding_stream(res, self.weight, ctx.token_ids, self.scale, ctx.error_flag)
+        return res, (res.clone() if keep else None)
 
 
 @register_part("embedding", "normed_token_embedding")

@@ -16,6 +16,10 @@ shared by all heads, a further `rope_dim` rows of the down projection that are n
 positions (halves paired, the first `rope_dims` values) and the score is scale * (q_plain . k_plain + q_rot . k_rot).
 The cached row is then [c | k_rot | zeros] and the query [Wuk^T q_plain | q_rot | zeros]: one dot product gives the
 whole score, and the row still serves as the value because the value expansion reads its first `rank` values only.
+`rope_interleaved` pairs neighbours instead of halves; `rope_scaling` ("yarn" and its constants) stretches the frequencies
+and multiplies cos and sin.
+`q_rank` > 0: the queries come through a low-rank vector too, q = (norm(h Wdq^T) * wq) Wuq^T; it rides in the merged down
+projection and one kernel norms both vectors of a token.
 `sink`: a learned number per head whose exponential joins the softmax's denominator without a key or a value.
 """
 from __future__ import annotations
@@ -29,6 +33,7 @@ from .. import kernels
 from .base import KVCacheSpec, LayerCache, Mixer, StepContext, WeightSpec, register_part
 from .attention import paged_attend
 from .linear import batched_matmul_tn, matmul_tn
+from .rope import rope_inverse_frequencies, yarn_magnitude
 
 USE_FAST_KERNELS = True     # bfloat16: the tensor-core attention kernels on the one-plane cache
 
@@ -39,7 +44,8 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, kv_rank: int, eps: float,
                  scale: Optional[float] = None, window: Optional[int] = None, gate: bool = True, rope_dim: int = 0,
-                 rope_dims: Optional[int] = None, rope_base: float = 10000.0, sink: bool = False):
+                 rope_dims: Optional[int] = None, rope_base: float = 10000.0, sink: bool = False, q_rank: int = 0,
+                 rope_interleaved: bool = False, rope_scaling: Optional[Dict[str, float]] = None):
         self.hidden_size, self.num_heads, self.head_dim, self.value_dim = int(hidden_size), int(num_heads), int(head_dim), int(value_dim)
         self.kv_rank = int(kv_rank)
         self.rope_dim = int(rope_dim or 0)
@@ -47,6 +53,12 @@ class LatentAttention(Mixer):
         if self.rope_dims % 2 or not (0 <= self.rope_dims <= self.rope_dim):
             raise ValueError(f"{self.rope_dims} rotated values of {self.rope_dim}: an even number, at most all of them")
         self.rope_base = float(rope_base)
+        # rope_scaling: {"factor", "original", "fast", "slow"} of the yarn kind
+        self.rope_interleaved, self.rope_scaling = bool(rope_interleaved), dict(rope_scaling) if rope_scaling else None
+        self.rope_mult = yarn_magnitude(float(self.rope_scaling["factor"])) if self.rope_scaling else 1.0
+        self.q_rank = int(q_rank or 0)
+        if self.q_rank and not self.rope_dim:
+            raise ValueError("a low-rank query goes with a rotated key part")
         self.has_sink = bool(sink)
         self.padded_rank = (self.kv_rank + self.rope_dim + 15) // 16 * 16
         if self.padded_rank > kernels.GENERIC_MAX_HEAD_DIM:
@@ -60,6 +72,9 @@ class LatentAttention(Mixer):
         self._sink32: Optional[torch.Tensor] = None
         self._inv_freq: Optional[torch.Tensor] = None
         self.qcg: Optional[torch.Tensor] = None
+        self.uq: Optional[torch.Tensor] = None
+        self.q_norm: Optional[torch.Tensor] = None
+        self._q_norm32: Optional[torch.Tensor] = None
         self.c_norm: Optional[torch.Tensor] = None
         self.uk: Optional[torch.Tensor] = None
         self.uv: Optional[torch.Tensor] = None
@@ -70,10 +85,13 @@ class LatentAttention(Mixer):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         D, R = self.hidden_size, self.kv_rank
-        merged = [(self.q_size, D), (R + self.rope_dim, D)] + ([(self.num_heads, D)] if self.has_gate else [])
+        merged = [(self.q_rank or self.q_size, D), (R + self.rope_dim, D)] + ([(self.num_heads, D)] if self.has_gate else [])
         specs = {"qcg": WeightSpec(merged), "c_norm": WeightSpec([(R,)], keep_fp32=True),
                  "uk": WeightSpec([(self.num_heads * self.head_dim, R)]), "uv": WeightSpec([(self.v_size, R)]),
                  "o": WeightSpec([(D, self.v_size)])}
+        if self.q_rank:
+            specs["uq"] = WeightSpec([(self.q_size, self.q_rank)])
+            specs["q_norm"] = WeightSpec([(self.q_rank,)], keep_fp32=True)
         if self.has_sink:
             specs["sink"] = WeightSpec([(self.num_heads,)], keep_fp32=True)
         return specs
@@ -82,7 +100,7 @@ class LatentAttention(Mixer):
         return KVCacheSpec(1, self.padded_rank, self.window, planes=1)
 
     def activation_width(self) -> int:
-        return self.q_size + self.kv_rank + self.rope_dim + self.num_heads + 2 * self.num_heads * self.padded_rank + self.v_size
+        return self.q_size + 2 * self.q_rank + self.kv_rank + self.rope_dim + self.num_heads + 2 * self.num_heads * self.padded_rank + self.v_size
 
     def prepare(self, dtype, device) -> None:
         if dtype == torch.bfloat16 and not kernels.mma_attention_supported(dtype, self.padded_rank):
@@ -99,9 +117,12 @@ class LatentAttention(Mixer):
         self._norm32 = self.c_norm.float().contiguous()
         self._sink32 = self.sink.float().contiguous() if self.has_sink else None
         if self.rope_dims:
-            n = self.rope_dims
-            self._inv_freq = torch.tensor([self.rope_base ** (-2.0 * i / n) for i in range(n // 2)],
+            sc = self.rope_scaling
+            kw = dict(scaling_type="yarn", factor=float(sc["factor"]), original_max_position_embeddings=sc["original"],
+                      beta_fast=float(sc["fast"]), beta_slow=float(sc["slow"])) if sc else {}
+            self._inv_freq = torch.tensor(rope_inverse_frequencies(self.rope_dims, self.rope_base, **kw),
                                           dtype=torch.float64).to(torch.float32).to(device)
+        self._q_norm32 = self.q_norm.float().contiguous() if self.q_rank else None
 
     def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
         H, dk, dv, R, Rp = self.num_heads, self.head_dim, self.value_dim, self.kv_rank, self.padded_rank
@@ -109,16 +130,22 @@ class LatentAttention(Mixer):
         group = ctx.groups[cache.group]
         dr = self.rope_dim
         p = matmul_tn(h, self.qcg)
-        q, c_raw = p[:, :self.q_size], p[:, self.q_size:self.q_size + R + dr]
-        g = p[:, self.q_size + R + dr:] if self.has_gate else None
+        c0 = self.q_rank or self.q_size                       # the columns before the key's vector: the query, or its vector
+        q, c_raw = p[:, :c0], p[:, c0:c0 + R + dr]
+        g = p[:, c0 + R + dr:] if self.has_gate else None
+        rot = dict(interleaved=self.rope_interleaved, rot_mult=self.rope_mult)
         qa = torch.empty((n, H * Rp), dtype=p.dtype, device=p.device)
         if dr:
-            if cache.owner:
+            cq = torch.empty((n, self.q_rank), dtype=p.dtype, device=p.device) if self.q_rank else None
+            if cache.owner or self.q_rank:
                 kernels.latent_norm_rope_cache_write(c_raw, self._norm32, self.eps, cache.kv, ctx.positions, ctx.token_seq,
                                                      group.block_table, group.block_size, R, dr, self.rope_dims,
-                                                     self._inv_freq, ctx.error_flag)
+                                                     self._inv_freq, ctx.error_flag, q_rank=self.q_rank, wq=self._q_norm32,
+                                                     q_out=cq, write=cache.owner, **rot)
+            if self.q_rank:
+                q = matmul_tn(cq, self.uq)
             batched_matmul_tn(qa.view(n, H, Rp)[:, :, :R], q.view(n, H, dk + dr)[:, :, :dk], self._uk_t)
-            kernels.latent_query_rope(qa, q, ctx.positions, H, dk, dr, self.rope_dims, self._inv_freq, R, Rp)
+            kernels.latent_query_rope(qa, q, ctx.positions, H, dk, dr, self.rope_dims, self._inv_freq, R, Rp, **rot)
         else:
             if cache.owner:
                 kernels.latent_norm_cache_write(c_raw, self._norm32, self.eps, cache.kv, ctx.positions, ctx.token_seq,

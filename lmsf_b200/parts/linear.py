@@ -32,12 +32,26 @@ def _skinny_takes(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def matmul_tn(x: Union[torch.Tensor, Prenormed], w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-              bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x [M, K] times w [N, K] transposed -> [M, N] in `out_dtype` (default: x's dtype), plus `bias` [N] if given
-    (added by a kernel of its own after the product, as the reference adds it: layers/linear.rs:100-104).  x may be a
-    `Prenormed`: the weight-streaming kernel divides its sums by the rows' root mean square."""
+              bias: Optional[torch.Tensor] = None, act: Optional[str] = None) -> torch.Tensor:
+    """x [M, K] times w [N, K] transposed -> [M, N] in `out_dtype` (default: x's dtype), plus `bias` [N] if given.  The
+    bfloat16 products add a bfloat16 bias to their float32 sums before they round (the reference adds it afterwards, in a
+    step of its own: layers/linear.rs:100-104); otherwise a kernel adds it after the product.  `act` "relu2": the square of
+    max(result, 0).  x may be a `Prenormed`: the weight-streaming kernel divides its sums by the rows' root mean square."""
+    plain = not isinstance(x, Prenormed)
+    hx = x if plain else x.x
+    fused_bias = bias if (bias is not None and bias.dtype == torch.bfloat16 and hx.dtype == torch.bfloat16) else None
+    dt = out_dtype or hx.dtype
+    if (fused_bias is not None or act is not None) and (bias is None or fused_bias is not None) and _skinny_takes(hx, w) and \
+            dt in (torch.bfloat16, torch.float32):
+        y = torch.empty((hx.shape[0], w.shape[0]), dtype=dt, device=w.device)
+        kernels.gemm_skinny(y, hx, w, prenorm=None if plain else (x.sumsq, x.eps, x.width), bias=fused_bias, act=act)
+        return y
+    if plain and fused_bias is not None and dt == torch.bfloat16:
+        y = torch.addmm(fused_bias, x, w.t())
+        if act is not None:
+            kernels.relu2_(y)
+        return y
     if isinstance(x, Prenormed):
-        dt = out_dtype or x.x.dtype
         if _skinny_takes(x.x, w) and dt in (torch.bfloat16, torch.float32):
             y = torch.empty((x.x.shape[0], w.shape[0]), dtype=dt, device=w.device)
             kernels.gemm_skinny(y, x.x, w, prenorm=(x.sumsq, x.eps, x.width))
@@ -47,6 +61,8 @@ def matmul_tn(x: Union[torch.Tensor, Prenormed], w: torch.Tensor, out_dtype: Opt
         y = _product_tn(x, w, out_dtype)
     if bias is not None:
         kernels.bias_add(y, bias if bias.dtype == y.dtype else bias.to(y.dtype))
+    if act is not None:
+        kernels.relu2_(y)
     return y
 
 

@@ -78,15 +78,16 @@ class GatedMLP(FeedForward):
 
 @register_part("feed_forward", "plain_mlp")
 class PlainMLP(FeedForward):
-    """A feed-forward without a gate: act(h Wu^T) Wd^T.  The one activation so far, `poly_norm`, is a polynomial whose powers
-    are each divided by their root mean square over the row of `intermediate_size` values:
+    """A feed-forward without a gate: act(h Wu^T) Wd^T.  `relu2` is the square of max(z, 0) (in a decode step part of the
+    product before it).  `poly_norm` is a polynomial whose powers are each divided by their root mean square over the row of
+    `intermediate_size` values:
         act(z) = a N(z) + b N(z^2) + c N(z^3) + e,   N(x) = x / sqrt(mean(x^2) + eps)
     with the four numbers (a, b, c, e) a weight of the part (`act`).  The sums and factors are float32 (csrc/activation.cu)."""
     graph_safe = True
 
-    def __init__(self, hidden_size: int, intermediate_size: int, eps: float, activation: str = "poly_norm"):
-        if activation != "poly_norm":
-            raise ValueError(f"activation {activation!r} is not supported by the plain feed-forward (known: poly_norm)")
+    def __init__(self, hidden_size: int, intermediate_size: int, eps: float = 1e-6, activation: str = "poly_norm"):
+        if activation not in ("poly_norm", "relu2"):
+            raise ValueError(f"activation {activation!r} is not supported by the plain feed-forward (known: poly_norm, relu2)")
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.eps, self.activation = float(eps), activation
         self.up: Optional[torch.Tensor] = None
@@ -95,17 +96,21 @@ class PlainMLP(FeedForward):
         self._coef: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        return {"up": WeightSpec([(self.intermediate_size, self.hidden_size)]),
-                "down": WeightSpec([(self.hidden_size, self.intermediate_size)]),
-                "act": WeightSpec([(4,)], keep_fp32=True)}
+        specs = {"up": WeightSpec([(self.intermediate_size, self.hidden_size)]),
+                 "down": WeightSpec([(self.hidden_size, self.intermediate_size)])}
+        if self.activation == "poly_norm":
+            specs["act"] = WeightSpec([(4,)], keep_fp32=True)
+        return specs
 
     def prepare(self, dtype, device) -> None:
-        self._coef = self.act.float().contiguous()
+        self._coef = self.act.float().contiguous() if self.activation == "poly_norm" else None
 
     def activation_width(self) -> int:
         return 2 * self.intermediate_size
 
     def forward(self, ctx: StepContext, h):
+        if self.activation == "relu2":
+            return matmul_tn(matmul_tn(h, self.up, act="relu2"), self.down)
         z = matmul_tn(h, self.up)
         m = torch.empty_like(z)
         kernels.poly_norm(m, z, self._coef, self.eps)

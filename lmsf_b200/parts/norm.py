@@ -36,7 +36,7 @@ class RMSNorm(Norm):
     def set_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
         super().set_weights(tensors)
         if self.weight_offset and "weight" in tensors:
-            self.weight = (tensors["weight"].float() + self.weight_offset).to(tensors["weight"].dtype)
+            self.weight = tensors["weight"].float() + self.weight_offset     # float32: the sum has more digits than the stored weight
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         specs = {"weight": WeightSpec([(self.hidden_size,)], keep_fp32=True)}

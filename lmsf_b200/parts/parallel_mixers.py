@@ -1,0 +1,79 @@
+"""Two mixers side by side that read the same input and whose outputs are added with a factor each:
+
+  out = left_scale * attention(h) + right_scale * memory(h)
+
+The left one is attention whose values are its keys, the right one a matrix memory.  Their matrices are merged when the weights
+are on the device: one product for everything that reads h (queries, keys, and the memory's q, k, v, gates), one for both
+output projections ([left | right] side by side).  The right factor is applied to the memory's float32 output before it is
+rounded; the left one is asked of the block (`Mixer.out_scale`), which adds the result to the float32 stream: nothing is
+rounded on its account.  The pages of the cache are the left mixer's, the state slot the right one's.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .base import KVCacheSpec, LayerCache, Mixer, StateSpec, StepContext, register_part
+from .linear import matmul_tn
+
+
+@register_part("mixer", "parallel_mixers")
+class ParallelMixers(Mixer):
+    graph_safe = True
+
+    def __init__(self, mixer_left: Mixer, mixer_right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0):
+        left, right = mixer_left, mixer_right
+        if not getattr(left, "values_are_keys", False) or not hasattr(right, "mix_projected") or left.hidden_size != right.hidden_size:
+            raise ValueError("side by side stand attention whose values are its keys (left) and a matrix memory (right) of one width")
+        if left.has_out_bias:
+            raise ValueError("mixers side by side are not built with a bias of the output projection")
+        self.left, self.right = left, right
+        self.left_scale, self.right_scale = float(left_scale), float(right_scale)
+        # the block multiplies by the left factor; a left factor of zero leaves the right mixer alone
+        self.out_scale = self.left_scale if self.left_scale != 0.0 else 1.0
+        self.right_factor = self.right_scale / self.out_scale
+        self._in: Optional[torch.Tensor] = None
+        self._in_bias: Optional[torch.Tensor] = None
+        self._out: Optional[torch.Tensor] = None
+        self.out_pad = 0
+
+    def cache_spec(self) -> Optional[KVCacheSpec]:
+        return self.left.cache_spec()
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return self.right.state_spec()
+
+    def activation_width(self) -> int:
+        return self.left.activation_width() + self.right.activation_width() + self.left.hidden_size
+
+    def prepare(self, dtype, device) -> None:
+        L, R = self.left, self.right
+        if self._in is not None and self._in.device == L.qkv.device and L.qkv.data_ptr() == self._in.data_ptr():
+            return
+        rows = L.qkv.shape[0] + R.in_proj.shape[0]
+        pad = -rows % 8                                    # row strides that are multiples of 16 bytes
+        self._in = torch.cat([L.qkv, R.in_proj, L.qkv.new_zeros((pad, L.qkv.shape[1]))], 0).contiguous()
+        self._in_bias = None
+        if L.qkv_bias is not None:
+            self._in_bias = torch.cat([L.qkv_bias, L.qkv_bias.new_zeros(rows + pad - L.qkv_bias.shape[0])], 0).contiguous()
+        left_o = L.o if self.left_scale != 0.0 else torch.zeros_like(L.o)
+        self.out_pad = -(L.o.shape[1] + R.o.shape[1]) % 8
+        self._out = torch.cat([left_o, R.o, L.o.new_zeros((L.o.shape[0], self.out_pad))], 1).contiguous()
+        # the parts' own matrices become views of the merged ones
+        n = L.qkv.shape[0]
+        L.qkv, R.in_proj = self._in[:n], self._in[n:rows]
+        if self.left_scale != 0.0:
+            L.o = self._out[:, :L.o.shape[1]]
+        R.o = self._out[:, L.o.shape[1]:L.o.shape[1] + R.o.shape[1]]
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
+        L, R = self.left, self.right
+        a, b = L.q_size, R.v_size
+        p, cached = L.project(ctx, h, self._in, self._in_bias, cache)
+        make = torch.zeros if self.out_pad else torch.empty
+        y = make((ctx.n_tokens, a + b + self.out_pad), dtype=p.dtype, device=p.device)
+        L.attend_projected(ctx, p, cached, cache, y[:, :a])
+        n = L.q_size + L.kv_size
+        R.mix_projected(ctx, p[:, n:n + R.in_size], cache, y[:, a:a + b], self.right_factor)
+        return matmul_tn(y, self._out)

@@ -15,16 +15,19 @@ from typing import List, Optional, Tuple
 import torch
 
 from .. import kernels
-from .base import PositionEncoding, StepContext, WeightSpec, register_part
+from .base import ANY_SIZE, PositionEncoding, StepContext, WeightSpec, register_part
 
 
 def rope_inverse_frequencies(rot_dim: int, theta: float, scaling_type: str = "default", factor: float = 1.0,
                              low_freq_factor: float = 1.0, high_freq_factor: float = 4.0,
-                             original_max_position_embeddings: int = 8192) -> List[float]:
+                             original_max_position_embeddings: int = 8192, beta_fast: float = 32.0,
+                             beta_slow: float = 1.0) -> List[float]:
     """f_i = theta^(-2i/rot_dim), then by scaling type:
     linear: f_i / factor.
     llama3: wavelength 2 pi / f_i shorter than L0/high keeps f_i, longer than L0/low gives f_i / factor,
-            between them an interpolation with s = (L0 / wavelength - low) / (high - low)."""
+            between them an interpolation with s = (L0 / wavelength - low) / (high - low).
+    yarn: pairs that turn more than beta_fast times within L0 positions keep f_i, pairs that turn less than beta_slow times
+            get f_i / factor, between them (counted in pairs) a linear ramp; `yarn_magnitude` goes with it."""
     inv = [theta ** (-(2.0 * i) / rot_dim) for i in range(rot_dim // 2)]
     if scaling_type == "default":
         return inv
@@ -43,7 +46,18 @@ def rope_inverse_frequencies(rot_dim: int, theta: float, scaling_type: str = "de
                 s = (l0 / wavelen - low_freq_factor) / (high_freq_factor - low_freq_factor)
                 out.append((1.0 - s) * f / factor + s * f)
         return out
+    if scaling_type == "yarn":
+        pair_of = lambda turns: rot_dim * math.log(original_max_position_embeddings / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+        lo = max(math.floor(pair_of(beta_fast)), 0)
+        hi = min(math.ceil(pair_of(beta_slow)), rot_dim - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(rot_dim // 2)]
+        return [f / factor * r + f * (1.0 - r) for f, r in zip(inv, ramp)]
     raise ValueError(f"unknown rope scaling type {scaling_type!r}")
+
+
+def yarn_magnitude(factor: float) -> float:
+    """What cos and sin are multiplied by where positions are stretched by `factor` the yarn way."""
+    return 0.1 * math.log(factor) + 1.0
 
 
 @register_part("position_encoding", "rotary")
@@ -135,3 +149,56 @@ class LogDistanceBias(PositionEncoding):
 
     def score_log_bias(self) -> Optional[Tuple[torch.Tensor, torch.Tensor]]:
         return self._r
+
+
+def distance_bucket(n: int, count: int, far: float) -> int:
+    """Which of `count` learned entries serves the distance n >= 0: the first half serve one distance each, the others ranges
+    that widen with the logarithm of the distance, the last one everything from `far` on."""
+    half = count // 2
+    if n < half:
+        return n
+    if half == 0 or far <= half:
+        return count - 1
+    return min(count - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (count - half)))
+
+
+@register_part("position_encoding", "bucketed_distance_bias")
+class BucketedDistanceBias(PositionEncoding):
+    """Positions enter the scores, not q and k: a learned number per (bucket of the distance, query head) is added to every
+    scaled score (weight `table` [buckets, heads]; see `distance_bucket`).  The attention kernels take it spread out over the
+    distances 0 .. far, float32 [heads, entries], whose last entry serves every larger distance.  `buckets` None: as many as
+    the stored table has rows."""
+    graph_safe = True
+
+    def __init__(self, num_heads: int, far: float, buckets: Optional[int] = None):
+        self.num_heads, self.far = int(num_heads), float(far)
+        self.buckets = int(buckets) if buckets is not None else None
+        if (self.buckets is not None and self.buckets < 1) or not self.far > 0:
+            raise ValueError(f"a distance bias of {buckets} buckets up to distance {far}")
+        self.table: Optional[torch.Tensor] = None
+        self._spread: Optional[torch.Tensor] = None
+
+    def weight_specs(self):
+        return {"table": WeightSpec([(self.buckets if self.buckets is not None else ANY_SIZE, self.num_heads)], keep_fp32=True)}
+
+    def set_weights(self, tensors) -> None:
+        super().set_weights(tensors)
+        if "table" in tensors:
+            self.buckets = int(self.table.shape[0])
+
+    def bucket_list(self) -> List[int]:
+        """The bucket of every distance up to the first that, with all larger ones, belongs to the last bucket."""
+        out = [distance_bucket(0, self.buckets, self.far)]
+        while out[-1] < self.buckets - 1:
+            out.append(distance_bucket(len(out), self.buckets, self.far))
+        return out
+
+    def prepare(self, dtype, device) -> None:
+        which = torch.tensor(self.bucket_list(), dtype=torch.long, device=self.table.device)
+        self._spread = self.table.float()[which].t().contiguous().to(device)
+
+    def apply(self, ctx, q, k, n_q_heads, n_kv_heads, head_dim) -> None:
+        return None
+
+    def score_distance_table(self) -> Optional[torch.Tensor]:
+        return self._spread

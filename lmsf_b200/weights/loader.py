@@ -57,13 +57,13 @@ def collect_requirements(model) -> List[Tuple[object, str, WeightSpec, List[str]
 def check_tensors(model, entries: Dict[str, TensorEntry], model_dir: str = "") -> None:
     missing, wrong, used = [], [], set()
     for _, _, wspec, names in collect_requirements(model):
-        for name, shape in zip(names, wspec.shapes):
+        for i, (name, shape) in enumerate(zip(names, wspec.shapes)):
             used.add(name)
             e = entries.get(name)
             if e is None:
                 if name not in missing:
                     missing.append(name)
-            elif tuple(e.shape) != tuple(shape):
+            elif not wspec.matches(i, e.shape):
                 wrong.append((name, shape, e.shape))
     ignored = [re.compile(p) for p in model.spec.ignored_weights]
     unexpected = sorted(n for n in entries if n not in used and not any(p.search(n) for p in ignored))

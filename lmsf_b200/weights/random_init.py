@@ -36,10 +36,10 @@ def tensor_list(model: DecoderModel) -> List[Tuple[str, Tuple[int, ...], bool]]:
     """(name, shape, is a norm-like vector) of every stored tensor of the model, once each."""
     seen, out = set(), []
     for _, _, wspec, names in collect_requirements(model):
-        for name, shape in zip(names, wspec.shapes):
+        for i, name in enumerate(names):
             if name not in seen:
                 seen.add(name)
-                out.append((name, tuple(shape), wspec.keep_fp32))
+                out.append((name, wspec.concrete(i), wspec.keep_fp32))
     return out
 
 
@@ -75,8 +75,8 @@ def init_random_on_device(model: DecoderModel, seed: int, dtype: torch.dtype, de
         key = tuple(names)
         t = done.get(key)
         if t is None:
-            rows = sum(s[0] for s in wspec.shapes)
-            shape = (rows, *wspec.shapes[0][1:])
+            sizes = [wspec.concrete(i) for i in range(len(wspec.shapes))]
+            shape = (sum(s[0] for s in sizes), *sizes[0][1:])
             if wspec.keep_fp32:
                 t = torch.ones(shape, dtype=dtype, device=device)
             else:
