@@ -6,7 +6,7 @@
 // vllm/kernels/attention/attention_kernels.cu:82-414.  Differences: one kernel serves prompt
 // portions and decoded tokens alike (every query token reads its keys from pages, its own key
 // included, which the cache write has stored before); the softmax is exact (no 1e-6 in the
-// denominator, expf rather than __expf); any head size that is a multiple of 16 up to 512.
+// denominator, expf rather than __expf); any head size that is a multiple of 16 up to 640.
 //
 // One block of 4 warps per (query token, query head).  Keys are walked in tiles of 32 that are
 // aligned to absolute positions; tile j belongs to warp j % 4; every warp keeps a running
@@ -19,7 +19,7 @@ LMSF_DEFINE_LAST_ERROR(lmsf_attention_generic)
 
 namespace lmsf {
 
-constexpr int kMaxHeadDim = 512;
+constexpr int kMaxHeadDim = 640;
 constexpr int kWarps = 4;
 
 struct GenericAttnArgs {
@@ -43,10 +43,11 @@ struct GenericAttnArgs {
   const float* dist; int dist_n;               // [n_q_heads][dist_n] or null: the entry of (query position - key position), the last for larger ones, is added
 };
 
-template <typename T>
+// MAXD: the largest head size of a build (accumulators in registers)
+template <typename T, int MAXD>
 __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericAttnArgs a) {
-  __shared__ float qs[kMaxHeadDim];
-  __shared__ float part_acc[kWarps][kMaxHeadDim];
+  __shared__ float qs[MAXD];
+  __shared__ float part_acc[kWarps][MAXD];
   __shared__ float part_m[kWarps], part_l[kWarps];
 
   const int t = blockIdx.x, head = blockIdx.y;
@@ -69,9 +70,9 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
   const int nd = (hd + 31) / 32;
 
   float m = -INFINITY, l = 0.f;
-  float acc[kMaxHeadDim / 32];
+  float acc[MAXD / 32];
 #pragma unroll
-  for (int i = 0; i < kMaxHeadDim / 32; ++i) acc[i] = 0.f;
+  for (int i = 0; i < MAXD / 32; ++i) acc[i] = 0.f;
 
   // tiles 0 .. (keep - 1) / 32 hold the kept first keys, tiles lo / 32 .. pos / 32 the window; tile j is always warp j % 4's
   const int first_tile = keep > 0 ? 0 : lo / 32;
@@ -107,7 +108,7 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
         if (rj < 0) continue;
         const T* vr = (const T*)a.cache + rj + v_off;
 #pragma unroll
-        for (int i = 0; i < kMaxHeadDim / 32; ++i) {
+        for (int i = 0; i < MAXD / 32; ++i) {
           const int d = lane + 32 * i;
           if (i < nd && d < hd) acc[i] = fmaf(pj, to_f32(vr[d]), acc[i]);
         }
@@ -120,14 +121,14 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
     const float alpha = expf(m - m_new);  // m = -inf on the first tile gives 0
     l = l * alpha + warp_sum(p);
 #pragma unroll
-    for (int i = 0; i < kMaxHeadDim / 32; ++i) acc[i] *= alpha;
+    for (int i = 0; i < MAXD / 32; ++i) acc[i] *= alpha;
     for (int j = 0; j < 32; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const long long rj = __shfl_sync(0xffffffffu, row, j);
       if (rj < 0) continue;  // same for the whole warp
       const T* vr = (const T*)a.cache + rj + v_off;
 #pragma unroll
-      for (int i = 0; i < kMaxHeadDim / 32; ++i) {
+      for (int i = 0; i < MAXD / 32; ++i) {
         const int d = lane + 32 * i;
         if (i < nd && d < hd) acc[i] = fmaf(pj, to_f32(vr[d]), acc[i]);
       }
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(kWarps * 32) attention_generic_kernel(GenericA
 
   if (lane == 0) { part_m[warp] = m; part_l[warp] = l; }
 #pragma unroll
-  for (int i = 0; i < kMaxHeadDim / 32; ++i) {
+  for (int i = 0; i < MAXD / 32; ++i) {
     const int d = lane + 32 * i;
     if (i < nd && d < hd) part_acc[warp][d] = acc[i];
   }
@@ -209,8 +210,12 @@ LMSF_API int lmsf_attention_generic_dist(const void* q, long long q_stride, void
   if (sigmoid && sinks) LMSF_REFUSE("attention: sinks belong to a softmax, not to sigmoid weights");
   dim3 grid(n_tokens, n_q_heads);
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == LMSF_F32) attention_generic_kernel<float><<<grid, kWarps * 32, 0, s>>>(a);
-  else attention_generic_kernel<bf16><<<grid, kWarps * 32, 0, s>>>(a);
+#define LMSF_GO(D) do { if (dtype == LMSF_F32) attention_generic_kernel<float, D><<<grid, kWarps * 32, 0, s>>>(a); \
+                        else attention_generic_kernel<bf16, D><<<grid, kWarps * 32, 0, s>>>(a); } while (0)
+  if (head_dim <= 128) LMSF_GO(128);
+  else if (head_dim <= 256) LMSF_GO(256);
+  else LMSF_GO(kMaxHeadDim);
+#undef LMSF_GO
   return LMSF_LAUNCH_STATUS();
 }
 

@@ -279,7 +279,7 @@ def qk_norm_rope_cache_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Opti
 
 # ----------------------------------------------------------------------------- attention (generic)
 
-GENERIC_MAX_HEAD_DIM = 512     # the plain attention kernel holds a head's accumulator in registers up to this size
+GENERIC_MAX_HEAD_DIM = 640     # the plain attention kernel holds a head's accumulator in registers up to this size
 
 
 def _per_head(t: Optional[torch.Tensor], heads: int, what: str) -> None:
