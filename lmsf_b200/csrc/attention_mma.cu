@@ -85,11 +85,12 @@ constexpr int kTableCache = 512;           // block-table entries of a split tha
 constexpr int kMergeWeights = 4096;        // (heads of a block) x splits whose weights fit the shared memory used for adding up
 
 // S: stages of the ring of key/value tiles (kStages; one more in the variant for launches of so few blocks that each
-// has an SM to itself, below)
-template <int W, int S = kStages>
+// has an SM to itself, below).  ONE: the cache's keys are its values; a stage then is half as large and S is twice as many.
+template <int W, int S = kStages, bool ONE = false>
 __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
   constexpr int kDecWarps = W, kDecThreads = 32 * W, kDecTile = 16 * W;
   using DSt = Stage<HD, kDecTile>;
+  constexpr int kStageBytes = ONE ? DSt::kBytes / 2 : DSt::kBytes;
   extern __shared__ __align__(16) unsigned char smem[];
   __shared__ int s_table[kTableCache];
   __shared__ int s_is_last;
@@ -175,11 +176,11 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
   const int safe_end = (ctx - 1) / kDecTile;                  // tiles below this index hold only older keys
   for (int s = 0; s < S - 1; ++s)
     if (s < n_tiles && tiles.at(tile_begin + s) < safe_end)
-      load_stage<HD, kDecTile, kDecThreads>(smem_base + s * DSt::kBytes, a.kv, table, kvh, tiles.at(tile_begin + s) * kDecTile, lo, ctx, table_off, keep);
+      load_stage<HD, kDecTile, kDecThreads, ONE>(smem_base + s * kStageBytes, a.kv, table, kvh, tiles.at(tile_begin + s) * kDecTile, lo, ctx, table_off, keep);
   pdl_wait();
   for (int s = 0; s < S - 1; ++s) {
     if (s < n_tiles && tiles.at(tile_begin + s) >= safe_end)
-      load_stage<HD, kDecTile, kDecThreads>(smem_base + s * DSt::kBytes, a.kv, table, kvh, tiles.at(tile_begin + s) * kDecTile, lo, ctx, table_off, keep);
+      load_stage<HD, kDecTile, kDecThreads, ONE>(smem_base + s * kStageBytes, a.kv, table, kvh, tiles.at(tile_begin + s) * kDecTile, lo, ctx, table_off, keep);
     cp_async_commit();
   }
 
@@ -209,11 +210,11 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
     {
       const int nxt = i + S - 1;
       if (nxt < n_tiles)
-        load_stage<HD, kDecTile, kDecThreads>(smem_base + (nxt % S) * DSt::kBytes, a.kv, table, kvh, tiles.at(tile_begin + nxt) * kDecTile, lo, ctx, table_off, keep);
+        load_stage<HD, kDecTile, kDecThreads, ONE>(smem_base + (nxt % S) * kStageBytes, a.kv, table, kvh, tiles.at(tile_begin + nxt) * kDecTile, lo, ctx, table_off, keep);
       cp_async_commit();
     }
-    const uint32_t kbase = smem_base + (i % S) * DSt::kBytes;       // this warp's rows are warp * 16 ..
-    const uint32_t vbase = kbase + kDecTile * DSt::kRowBytes;
+    const uint32_t kbase = smem_base + (i % S) * kStageBytes;       // this warp's rows are warp * 16 ..
+    const uint32_t vbase = ONE ? kbase : kbase + kDecTile * DSt::kRowBytes;
     const int key0 = tiles.at(tile_begin + i) * kDecTile + warp * 16;   // first key of this warp's 16
     if (key0 >= ctx || (key0 + 16 <= lo && key0 >= keep)) continue;     // nothing valid (uniform over the warp)
 
@@ -531,17 +532,21 @@ static int decode_smem_bytes(int group, int warps, int stages = lmsf::fa::kStage
 // The decode kernel of a width is allowed as much dynamic shared memory as the largest request so far: the attribute is
 // only ever raised (a query for a small group of heads must not lower what a launch for a large group was given).
 typedef void (*DecodeKernel)(lmsf::fa::DecodeArgs);
-static DecodeKernel decode_variant(int warps, bool deep) {
+static DecodeKernel decode_variant(int warps, bool deep, bool one = false) {
   using namespace lmsf::fa;
+  if (one) {      // the same shared memory, twice the stages of half the size
+    if (warps == 2) return decode_kernel<2, 2 * kStages, true>;
+    return deep ? (DecodeKernel)decode_kernel<4, 2 * kDeepStages, true> : (DecodeKernel)decode_kernel<4, 2 * kStages, true>;
+  }
   if (warps == 2) return decode_kernel<2>;
   return deep ? (DecodeKernel)decode_kernel<4, kDeepStages> : (DecodeKernel)decode_kernel<4>;
 }
 
-static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false) {
-  static int allowed[3] = {0, 0, 0};
-  const int v = warps == 2 ? 0 : (deep ? 2 : 1);
+static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false, bool one = false) {
+  static int allowed[6] = {0, 0, 0, 0, 0, 0};
+  const int v = (warps == 2 ? 0 : (deep ? 2 : 1)) + (one ? 3 : 0);
   if (smem <= allowed[v]) return cudaSuccess;
-  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep, one), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e == cudaSuccess) allowed[v] = smem;
   return e;
 }
@@ -686,9 +691,10 @@ static int decode_launch(lmsf::fa::DecodeArgs& a, int gy, int grid_x, int grid_z
     const long long clusters = (long long)gy * grid_z * (a.cluster ? 1 : grid_x);
     deep = fit[cs][R] > 0 && clusters <= fit[cs][R];
   }
-  DecodeKernel kernel = decode_variant(warps, deep);
+  const bool one = a.kv.v_off == 0;                        // keys that are values
+  DecodeKernel kernel = decode_variant(warps, deep, one);
   const int smem = decode_smem_bytes(a.group, warps, deep ? kDeepStages : kStages);
-  if (const cudaError_t e = decode_allow_smem(warps, smem, deep)) return (int)e;
+  if (const cudaError_t e = decode_allow_smem(warps, smem, deep, one)) return (int)e;
   if (!a.cluster) return launch_pdl(kernel, dim3(grid_x, (unsigned)gy, grid_z), dim3(32 * warps), smem, s, a);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(grid_x, (unsigned)gy, grid_z);

@@ -113,7 +113,8 @@ __device__ __forceinline__ float log_distance_bias2f(float r1, float r2, float d
   return r1 * __log2f(fmaf(r2, fmaxf(distance, 0.f), 1.0f));
 }
 
-// Shared-memory stage: TILE rows of K then TILE rows of V.  Every row carries 16 bytes of padding, which
+// Shared-memory stage: TILE rows of K then TILE rows of V (a cache whose keys are its values: TILE rows that serve as both, so
+// that the same memory holds twice the stages).  Every row carries 16 bytes of padding, which
 // makes the 8 rows of an ldmatrix fall into different banks for any HD.  Head size 64 is the exception: its rows
 // are exactly 128 bytes and the 16-byte chunk c of row r sits at chunk c ^ (r & 7) instead, so that a stage is 16 KB
 // and three stages leave room for four blocks on an SM (at head size 128 the same layout was measured slower than
@@ -134,7 +135,8 @@ template <int HD, int TILE = kTileKeys> struct Stage {
 // A thread copies one 16-byte column of several CONSECUTIVE rows, so that it looks its page up once per
 // page rather than once per row; a warp's copies of one pass cover whole rows (coalesced).
 // `table` may be a copy of a slice of the request's block table: entry i of it is block i + table_off.
-template <int HD, int TILE = kTileKeys, int THREADS = kThreads>
+// ONE: the cache holds one vector per token and head; no V half is written.
+template <int HD, int TILE = kTileKeys, int THREADS = kThreads, bool ONE = false>
 __device__ __forceinline__ void load_stage(uint32_t stage_base, const PagedKV& kv, const int* __restrict__ table, int kvh,
                                            int key0, int lo, int hi, int table_off = 0, int keep = 0) {
   using S = Stage<HD, TILE>;
@@ -160,7 +162,7 @@ __device__ __forceinline__ void load_stage(uint32_t stage_base, const PagedKV& k
       const bf16* src = ok ? page_ptr + (size_t)slot * HD : kv.cache;
       const uint32_t dst = stage_base + S::off(row, c);
       cp_async_16(dst, src, ok ? 16 : 0);
-      cp_async_16(dst + TILE * S::kRowBytes, ok ? src + v_off : src, ok ? 16 : 0);
+      if (!ONE) cp_async_16(dst + TILE * S::kRowBytes, ok ? src + v_off : src, ok ? 16 : 0);
     }
   } else {
     static_assert((TILE * S::kChunks) % THREADS == 0, "a stage's copies must divide evenly among the threads");
@@ -180,7 +182,7 @@ __device__ __forceinline__ void load_stage(uint32_t stage_base, const PagedKV& k
       }
       const uint32_t dst = stage_base + S::off(row, c);
       cp_async_16(dst, src, bytes);
-      cp_async_16(dst + TILE * S::kRowBytes, bytes ? src + v_off : src, bytes);
+      if (!ONE) cp_async_16(dst + TILE * S::kRowBytes, bytes ? src + v_off : src, bytes);
     }
   }
 }

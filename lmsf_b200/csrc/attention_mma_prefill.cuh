@@ -19,7 +19,10 @@ struct PrefillArgs {
 
 // One block: 64 query tokens (16 per warp) of one head.  Query i of a portion of n tokens of a request
 // that holds ctx keys after this step sits at position ctx - n + i and sees keys lo..position.
+// ONE: the cache's keys are its values; a stage is half as large and there are twice as many.
+template <bool ONE>
 __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
+  constexpr int S = ONE ? 2 * kStages : kStages, kStageBytes = ONE ? St::kBytes / 2 : St::kBytes;
   extern __shared__ __align__(16) unsigned char smem[];
   // blocks start in the order (all heads of tile 0, all heads of tile 1, ...); the caller lists the tiles that
   // see the most keys first
@@ -68,8 +71,8 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   const TileRange tiles = tile_range(lo, hi, keep, kTileKeys);
   const int n_tiles = tiles.n;
   const uint32_t smem_base = smem_u32(smem);
-  for (int s = 0; s < kStages - 1; ++s) {
-    if (s < n_tiles) load_stage<HD>(smem_base + s * St::kBytes, a.kv, table, kvh, tiles.at(s) * kTileKeys, lo, hi, 0, keep);
+  for (int s = 0; s < S - 1; ++s) {
+    if (s < n_tiles) load_stage<HD, kTileKeys, kThreads, ONE>(smem_base + s * kStageBytes, a.kv, table, kvh, tiles.at(s) * kTileKeys, lo, hi, 0, keep);
     cp_async_commit();
   }
 
@@ -81,18 +84,18 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   const float sl2 = a.scale * kLog2e;
 
   for (int i = 0; i < n_tiles; ++i) {
-    cp_async_wait<kStages - 2>();
+    cp_async_wait<S - 2>();
     __syncthreads();
     {
-      const int nxt = i + kStages - 1;
+      const int nxt = i + S - 1;
       if (nxt < n_tiles)
-        load_stage<HD>(smem_base + (nxt % kStages) * St::kBytes, a.kv, table, kvh, tiles.at(nxt) * kTileKeys, lo, hi, 0, keep);
+        load_stage<HD, kTileKeys, kThreads, ONE>(smem_base + (nxt % S) * kStageBytes, a.kv, table, kvh, tiles.at(nxt) * kTileKeys, lo, hi, 0, keep);
       cp_async_commit();
     }
     const int key0 = tiles.at(i) * kTileKeys;
     if (key0 > warp_last_pos || (key0 + kTileKeys <= warp_lo && key0 >= keep)) continue;   // all masked for this warp
-    const uint32_t kbase = smem_base + (i % kStages) * St::kBytes;
-    const uint32_t vbase = kbase + kTileKeys * St::kRowBytes;
+    const uint32_t kbase = smem_base + (i % S) * kStageBytes;
+    const uint32_t vbase = ONE ? kbase : kbase + kTileKeys * St::kRowBytes;
 
     float s[8][4];
 #pragma unroll
@@ -215,12 +218,14 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
   if (dist && dist_n <= 0) LMSF_REFUSE("attention_prefill: a table of %d distances", dist_n);
   a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   const int smem = kStages * St::kBytes;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const bool one = kv_planes == 1;
+  void (*kernel)(PrefillArgs) = one ? prefill_kernel<true> : prefill_kernel<false>;
+  static bool configured[2] = {false, false};
+  if (!configured[one]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    configured = true;
+    configured[one] = true;
   }
-  prefill_kernel<<<dim3(n_q_heads, n_tiles), kThreads, smem, (cudaStream_t)stream>>>(a);
+  kernel<<<dim3(n_q_heads, n_tiles), kThreads, smem, (cudaStream_t)stream>>>(a);
   return LMSF_LAUNCH_STATUS();
 }
