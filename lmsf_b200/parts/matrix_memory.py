@@ -21,7 +21,7 @@ from .. import kernels
 from .base import LayerCache, Mixer, StateSpec, StepContext, WeightSpec, register_part
 from .linear import matmul_tn
 
-LONG_PORTION = 96      # tokens from which a request's portion is cut into chunks that run in parallel
+LONG_PORTION = 64      # tokens from which a request's portion is cut into chunks that run in parallel
 
 
 @register_part("mixer", "matrix_memory")
