@@ -135,7 +135,7 @@ def kernels_alone(pk, width=4096, heads=32, kv_heads=8, dim=128, window=1024, mh
     kernels_attention(rec, tm, rnd, ints, pos, seq, cu, ctxl, cud, ctxd, flag, T, B, H, G, dim, window)
     # ---- the products of a decode step
     x8 = rnd(8, width)
-    extra = 2 * QK + 2 * V + 2 * mh
+    extra = (2 * QK + 2 * V + 2 * mh + 15) // 16 * 16
     Wm, bias = rnd((H + G) * dim + extra, width, scale=0.02), rnd((H + G) * dim + extra)
     pages = 64
     c1, c2 = torch.zeros(pages, 1, G, bs, dim, dtype=bf, device=dev), torch.zeros(pages, 2, G, bs, dim, dtype=bf, device=dev)

@@ -86,7 +86,8 @@ constexpr int kMergeWeights = 4096;        // (heads of a block) x splits whose 
 
 // S: stages of the ring of key/value tiles (kStages; one more in the variant for launches of so few blocks that each
 // has an SM to itself, below).  ONE: the cache's keys are its values; a stage then is half as large and S is twice as many.
-template <int W, int S = kStages, bool ONE = false>
+// TABLE: a table of distances is added to the scores (a build of its own: the test alone cost decode steps of the others 1 to 4 %).
+template <int W, int S = kStages, bool ONE = false, bool TABLE = false>
 __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
   constexpr int kDecWarps = W, kDecThreads = 32 * W, kDecTile = 16 * W;
   using DSt = Stage<HD, kDecTile>;
@@ -134,7 +135,7 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
       if (g4 + h * 8 < n_heads) { r1[h] = a.x.r1[head0 + g4 + h * 8]; r2[h] = a.x.r2[head0 + g4 + h * 8]; }
   }
   const float* dist_row[2] = {a.x.dist, a.x.dist};             // the heads' rows of a table of distances, if there is one
-  if (a.x.dist) {
+  if (TABLE) {
 #pragma unroll
     for (int h = 0; h < 2; ++h)
       if (g4 + h * 8 < n_heads) dist_row[h] = a.x.dist + (size_t)(head0 + g4 + h * 8) * a.x.dist_n;
@@ -237,7 +238,7 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
         const bool ok = (key >= lo || key < keep) && key < ctx;
         float v = ok ? fmaf(s[j][e], sl2, hb2[e >> 1]) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2(r1[e >> 1], r2[e >> 1], ctx - 1 - key);
-        if (dist_row[0] && ok) v += table_bias2(dist_row[e >> 1], a.x.dist_n, ctx - 1 - key);
+        if (TABLE && ok) v += table_bias2(dist_row[e >> 1], a.x.dist_n, ctx - 1 - key);
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -532,8 +533,16 @@ static int decode_smem_bytes(int group, int warps, int stages = lmsf::fa::kStage
 // The decode kernel of a width is allowed as much dynamic shared memory as the largest request so far: the attribute is
 // only ever raised (a query for a small group of heads must not lower what a launch for a large group was given).
 typedef void (*DecodeKernel)(lmsf::fa::DecodeArgs);
-static DecodeKernel decode_variant(int warps, bool deep, bool one = false) {
+static DecodeKernel decode_variant(int warps, bool deep, bool one = false, bool table = false) {
   using namespace lmsf::fa;
+  if (table && one) {
+    if (warps == 2) return decode_kernel<2, 2 * kStages, true, true>;
+    return deep ? (DecodeKernel)decode_kernel<4, 2 * kDeepStages, true, true> : (DecodeKernel)decode_kernel<4, 2 * kStages, true, true>;
+  }
+  if (table) {    // (without the deep ring)
+    if (warps == 2) return decode_kernel<2, kStages, false, true>;
+    return decode_kernel<4, kStages, false, true>;
+  }
   if (one) {      // the same shared memory, twice the stages of half the size
     if (warps == 2) return decode_kernel<2, 2 * kStages, true>;
     return deep ? (DecodeKernel)decode_kernel<4, 2 * kDeepStages, true> : (DecodeKernel)decode_kernel<4, 2 * kStages, true>;
@@ -542,11 +551,11 @@ static DecodeKernel decode_variant(int warps, bool deep, bool one = false) {
   return deep ? (DecodeKernel)decode_kernel<4, kDeepStages> : (DecodeKernel)decode_kernel<4>;
 }
 
-static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false, bool one = false) {
-  static int allowed[6] = {0, 0, 0, 0, 0, 0};
-  const int v = (warps == 2 ? 0 : (deep ? 2 : 1)) + (one ? 3 : 0);
+static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false, bool one = false, bool table = false) {
+  static int allowed[12] = {0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0};
+  const int v = (warps == 2 ? 0 : (deep ? 2 : 1)) + (one ? 3 : 0) + (table ? 6 : 0);
   if (smem <= allowed[v]) return cudaSuccess;
-  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep, one), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep, one, table), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e == cudaSuccess) allowed[v] = smem;
   return e;
 }
@@ -691,10 +700,11 @@ static int decode_launch(lmsf::fa::DecodeArgs& a, int gy, int grid_x, int grid_z
     const long long clusters = (long long)gy * grid_z * (a.cluster ? 1 : grid_x);
     deep = fit[cs][R] > 0 && clusters <= fit[cs][R];
   }
-  const bool one = a.kv.v_off == 0;                        // keys that are values
-  DecodeKernel kernel = decode_variant(warps, deep, one);
+  const bool one = a.kv.v_off == 0, table = a.x.dist != nullptr;      // keys that are values; a table of distances
+  if (table && !one) deep = false;
+  DecodeKernel kernel = decode_variant(warps, deep, one, table);
   const int smem = decode_smem_bytes(a.group, warps, deep ? kDeepStages : kStages);
-  if (const cudaError_t e = decode_allow_smem(warps, smem, deep, one)) return (int)e;
+  if (const cudaError_t e = decode_allow_smem(warps, smem, deep, one, table)) return (int)e;
   if (!a.cluster) return launch_pdl(kernel, dim3(grid_x, (unsigned)gy, grid_z), dim3(32 * warps), smem, s, a);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(grid_x, (unsigned)gy, grid_z);

@@ -19,8 +19,9 @@ struct PrefillArgs {
 
 // One block: 64 query tokens (16 per warp) of one head.  Query i of a portion of n tokens of a request
 // that holds ctx keys after this step sits at position ctx - n + i and sees keys lo..position.
-// ONE: the cache's keys are its values; a stage is half as large and there are twice as many.
-template <bool ONE>
+// ONE: the cache's keys are its values; a stage is half as large and there are twice as many.  TABLE: a table of distances is
+// added to the scores.
+template <bool ONE, bool TABLE>
 __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   constexpr int S = ONE ? 2 * kStages : kStages, kStageBytes = ONE ? St::kBytes / 2 : St::kBytes;
   extern __shared__ __align__(16) unsigned char smem[];
@@ -52,7 +53,7 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   const int keep = a.x.keep_first;                               // keys below it are seen behind the window too
   const bool sig = a.x.sigmoid != 0;
   const float hb2 = a.x.head_bias ? a.x.head_bias[head] * kLog2e : 0.f;
-  const float* dist_row = a.x.dist ? a.x.dist + (size_t)head * a.x.dist_n : nullptr;
+  const float* dist_row = TABLE ? a.x.dist + (size_t)head * a.x.dist_n : nullptr;
   const int warp_last_pos = start + q0 + min(warp * 16 + 15, rows_valid - 1);
   const int warp_first_pos = start + q0 + min(warp * 16, rows_valid - 1);
   const int warp_lo = first_seen(warp_first_pos, a.window, a.x.chunk);
@@ -122,7 +123,7 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
         const bool ok = key <= pos[h] && (key >= row_lo[h] || key < keep);
         float v = ok ? fmaf(s[j][e], sl2, hb2) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2f(r1, r2, dist0[h] - (float)(j * 8 + (e & 1)));
-        if (dist_row && ok) v += table_bias2(dist_row, a.x.dist_n, pos[h] - key);
+        if (TABLE && ok) v += table_bias2(dist_row, a.x.dist_n, pos[h] - key);
         s[j][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -219,12 +220,14 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
   a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
   const int smem = kStages * St::kBytes;
   const bool one = kv_planes == 1;
-  void (*kernel)(PrefillArgs) = one ? prefill_kernel<true> : prefill_kernel<false>;
-  static bool configured[2] = {false, false};
-  if (!configured[one]) {
+  const bool table = dist != nullptr;
+  void (*kernel)(PrefillArgs) = table ? (one ? prefill_kernel<true, true> : prefill_kernel<false, true>)
+                                      : (one ? prefill_kernel<true, false> : prefill_kernel<false, false>);
+  static bool configured[2][2] = {{false, false}, {false, false}};
+  if (!configured[table][one]) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    configured[one] = true;
+    configured[table][one] = true;
   }
   kernel<<<dim3(n_q_heads, n_tiles), kThreads, smem, (cudaStream_t)stream>>>(a);
   return LMSF_LAUNCH_STATUS();

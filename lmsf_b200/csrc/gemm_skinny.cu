@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
   auto issue_w = [&](int c) {
     const uint32_t st = ring + (c % STAGES) * kStage;
     const int k0 = (c_begin + c * c_stride) * kChunkK;
-    if (ROPE) issue_rows<16>(st, a.w + (size_t)f0 * a.ldw, a.ldw, pair8 ? 16 : min(16, a.N - f0), k0, a.K, lane, hi_off);
+    if (ROPE) issue_rows<16>(st, a.w + (size_t)f0 * a.ldw, a.ldw, 16, k0, a.K, lane, hi_off);
     else if (PAIR) issue_rows<16>(st, a.w + (size_t)n0 * a.ldw, a.ldw, min(8, rows_total - n0), k0, a.K, lane, a.up_offset - 8, true);
     else issue_rows<16>(st, a.w + (size_t)n0 * a.ldw, a.ldw, rows_total - n0, k0, a.K, lane);
     if (GROUPS == 2)
@@ -299,10 +299,10 @@ __global__ void __launch_bounds__(kWarps * 32) skinny_kernel(Args a) {
         sum += reinterpret_cast<const float*>(smem + w * (STAGES * kStage))[row * (8 * NT) + m];
       sum *= factor(m);
       const int n = row < 8 ? f0 + row : f1 + row - 8;                  // feature among q, k, v (and the rows behind them)
-      if (a.bias && n < a.N) sum += __bfloat162float(a.bias[n]);
+      if (a.bias) sum += __bfloat162float(a.bias[n]);
       const float val = __bfloat162float(__float2bfloat16_rn(sum));      // what the plain product would have stored
       const float other = __shfl_xor_sync(0xffffffffu, val, pair8 ? 8 : 1);
-      if (m >= a.M || n >= a.N) continue;
+      if (m >= a.M) continue;
       const int d = n % a.head_dim;
       const bool is_v = n >= q_size + kv_size;
       if (n >= q_size + a.planes * kv_size) {                            // a row that only passes: its own column of out
@@ -537,7 +537,7 @@ LMSF_API int lmsf_gemm_skinny_residual(void* out, long long ldo, const void* x, 
 // positions[m] of request token_seq[m].  inv_freq: [rot_dim / 2] float32 or null (no rotation).  Results are those
 // of lmsf_gemm_skinny (bfloat16 out) followed by the rotary / cache-write kernel, bit for bit.  in_sumsq, bias: as there.
 // planes = 1: there are no v rows (the cache holds one vector per token and kv head, key and value at once).  n_extra: w has
-// so many rows behind q, k and v whose results go to their own columns of q_out, a row of which then spans all of w's rows.
+// so many rows (a multiple of 16) behind q, k and v whose results go to their own columns of q_out, a row of which then spans all of w's rows.
 LMSF_API int lmsf_gemm_skinny_qkv_rope(void* q_out, long long ldq, const void* x, long long ldx, const void* w, long long ldw,
                                        int M, int K, const int* positions, const int* token_seq, const int* block_table,
                                        int max_blocks, int block_size, void* cache, long long page_stride,
@@ -560,8 +560,8 @@ LMSF_API int lmsf_gemm_skinny_qkv_rope(void* q_out, long long ldq, const void* x
     LMSF_REFUSE("gemm_skinny_qkv_rope: bad q or cache geometry");
   Args a{};
   a.x = (const bf16*)x; a.ldx = ldx; a.w = (const bf16*)w; a.ldw = ldw; a.out = q_out; a.ldo = ldq;
-  if ((planes != 1 && planes != 2) || n_extra < 0 || (n_extra > 0 && ldq < (long long)(n_q_heads + planes * n_kv_heads) * head_dim + n_extra))
-    LMSF_REFUSE("gemm_skinny_qkv_rope: planes=%d, %d rows behind them (an output row must hold every row of w then)", planes, n_extra);
+  if ((planes != 1 && planes != 2) || n_extra < 0 || n_extra % 16 || (n_extra > 0 && ldq < (long long)(n_q_heads + planes * n_kv_heads) * head_dim + n_extra))
+    LMSF_REFUSE("gemm_skinny_qkv_rope: planes=%d, %d rows behind them (a multiple of 16; an output row must hold every row of w then)", planes, n_extra);
   a.M = M; a.N = (n_q_heads + planes * n_kv_heads) * head_dim + n_extra; a.K = K; a.act = -1;
   a.bias = (const bf16*)bias; a.planes = planes;
   a.positions = positions; a.token_seq = token_seq; a.block_table = block_table; a.max_blocks = max_blocks;

@@ -538,7 +538,7 @@ def gemm_skinny_qkv_rope(q_out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, 
     with the rotary encoding and the cache write in its epilogue: q_out [M, heads * head_dim] gets the rotated q, the
     pages of `cache` the rotated k and v.  The same values as gemm_skinny followed by rope_cache_write.  prenorm, bias: as in
     `gemm_skinny`.  kv_planes 1: w has no v rows and the cache is [pages, 1, ...] (keys that are values).  n_extra: w has so
-    many rows behind them, whose results go to their own columns of q_out, [M, rows of w] then."""
+    many rows (a multiple of 16) behind them, whose results go to their own columns of q_out, [M, rows of w] then."""
     M, K = x.shape
     if (not gemm_skinny_qkv_rope_supported(x, w, head_dim, rot_dim if inv_freq is not None else 0, is_neox)
             or w.shape != ((n_q_heads + kv_planes * n_kv_heads) * head_dim + n_extra, K)

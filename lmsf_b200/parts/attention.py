@@ -218,7 +218,7 @@ class PagedAttention(Mixer):
         columns of the product are then not set)."""
         hx = h.x if isinstance(h, Prenormed) else h
         n_extra = w.shape[0] - self.q_size - self.kv_size
-        if (FUSE_QKV_ROPE and cache.owner and linear.USE_SKINNY and self._no_rotation()
+        if (FUSE_QKV_ROPE and cache.owner and linear.USE_SKINNY and self._no_rotation() and n_extra % 16 == 0
                 and kernels.gemm_skinny_qkv_rope_supported(hx, w, self.head_dim, 0, True)):
             group = ctx.groups[cache.group]
             p = torch.empty((ctx.n_tokens, w.shape[0] if n_extra else self.q_size), dtype=hx.dtype, device=hx.device)

@@ -52,7 +52,7 @@ class ParallelMixers(Mixer):
         if self._in is not None and self._in.device == L.qkv.device and L.qkv.data_ptr() == self._in.data_ptr():
             return
         rows = L.qkv.shape[0] + R.in_proj.shape[0]
-        pad = -rows % 8                                    # row strides that are multiples of 16 bytes
+        pad = -rows % 16                                   # what the weight-streaming product with a cache write takes
         self._in = torch.cat([L.qkv, R.in_proj, L.qkv.new_zeros((pad, L.qkv.shape[1]))], 0).contiguous()
         self._in_bias = None
         if L.qkv_bias is not None:
