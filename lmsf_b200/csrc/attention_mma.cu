@@ -87,7 +87,8 @@ constexpr int kMergeWeights = 4096;        // (heads of a block) x splits whose 
 // S: stages of the ring of key/value tiles (kStages; one more in the variant for launches of so few blocks that each
 // has an SM to itself, below).  ONE: the cache's keys are its values; a stage then is half as large and S is twice as many.
 // TABLE: a table of distances is added to the scores (a build of its own: the test alone cost decode steps of the others 1 to 4 %).
-template <int W, int S = kStages, bool ONE = false, bool TABLE = false>
+// CAP: scores are capped smoothly (a build of its own as well).
+template <int W, int S = kStages, bool ONE = false, bool TABLE = false, bool CAP = false>
 __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
   constexpr int kDecWarps = W, kDecThreads = 32 * W, kDecTile = 16 * W;
   using DSt = Stage<HD, kDecTile>;
@@ -203,7 +204,9 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
   float o[HD / 8][4];
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  const float sl2 = a.scale * kLog2e;
+  // a cap: the products enter tanh as s * scale / cap and leave it in base-2 units times cap * log2(e)
+  const float cap_in = CAP ? a.scale / a.x.softcap : 0.f;
+  const float sl2 = CAP ? a.x.softcap * kLog2e : a.scale * kLog2e;
 
   for (int i = 0; i < n_tiles; ++i) {
     cp_async_wait<S - 2>();
@@ -236,6 +239,7 @@ __global__ void __launch_bounds__(32 * W) decode_kernel(DecodeArgs a) {
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + j * 8 + t4 * 2 + (e & 1);
         const bool ok = (key >= lo || key < keep) && key < ctx;
+        if (CAP) s[j][e] = tanh_score(s[j][e] * cap_in);
         float v = ok ? fmaf(s[j][e], sl2, hb2[e >> 1]) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2(r1[e >> 1], r2[e >> 1], ctx - 1 - key);
         if (TABLE && ok) v += table_bias2(dist_row[e >> 1], a.x.dist_n, ctx - 1 - key);
@@ -533,8 +537,12 @@ static int decode_smem_bytes(int group, int warps, int stages = lmsf::fa::kStage
 // The decode kernel of a width is allowed as much dynamic shared memory as the largest request so far: the attribute is
 // only ever raised (a query for a small group of heads must not lower what a launch for a large group was given).
 typedef void (*DecodeKernel)(lmsf::fa::DecodeArgs);
-static DecodeKernel decode_variant(int warps, bool deep, bool one = false, bool table = false) {
+static DecodeKernel decode_variant(int warps, bool deep, bool one = false, bool table = false, bool cap = false) {
   using namespace lmsf::fa;
+  if (cap) {      // keys and values, no table
+    if (warps == 2) return decode_kernel<2, kStages, false, false, true>;
+    return deep ? (DecodeKernel)decode_kernel<4, kDeepStages, false, false, true> : (DecodeKernel)decode_kernel<4, kStages, false, false, true>;
+  }
   if (table && one) {
     if (warps == 2) return decode_kernel<2, 2 * kStages, true, true>;
     return deep ? (DecodeKernel)decode_kernel<4, 2 * kDeepStages, true, true> : (DecodeKernel)decode_kernel<4, 2 * kStages, true, true>;
@@ -551,11 +559,11 @@ static DecodeKernel decode_variant(int warps, bool deep, bool one = false, bool 
   return deep ? (DecodeKernel)decode_kernel<4, kDeepStages> : (DecodeKernel)decode_kernel<4>;
 }
 
-static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false, bool one = false, bool table = false) {
-  static int allowed[12] = {0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0};
-  const int v = (warps == 2 ? 0 : (deep ? 2 : 1)) + (one ? 3 : 0) + (table ? 6 : 0);
+static cudaError_t decode_allow_smem(int warps, int smem, bool deep = false, bool one = false, bool table = false, bool cap = false) {
+  static int allowed[15] = {0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0, 0};
+  const int v = (warps == 2 ? 0 : (deep ? 2 : 1)) + (cap ? 12 : (one ? 3 : 0) + (table ? 6 : 0));
   if (smem <= allowed[v]) return cudaSuccess;
-  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep, one, table), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const cudaError_t e = cudaFuncSetAttribute(decode_variant(warps, deep, one, table, cap), cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e == cudaSuccess) allowed[v] = smem;
   return e;
 }
@@ -639,7 +647,7 @@ LMSF_API int lmsf_attention_decode_width(const void* q, long long q_stride, void
                                          int n_q_heads, int head_dim, int n_splits, int block_warps, void* scratch,
                                          int kv_planes, int chunk, const float* r1, const float* r2, const float* sinks,
                                          int keep_first, int sigmoid, const float* head_bias, const float* dist, int dist_n,
-                                         void* stream) {
+                                         float softcap, void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (n_served <= 0) return 0;
@@ -670,7 +678,7 @@ LMSF_API int lmsf_attention_decode_width(const void* q, long long q_stride, void
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_decode: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_decode: sinks belong to a softmax, not to sigmoid weights");
   if (dist && dist_n <= 0) LMSF_REFUSE("attention_decode: a table of %d distances", dist_n);
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n, softcap > 0.f ? softcap : 0.f};
   a.rows = decode_rows(group);
   if (block_warps != 0 && block_warps != 2 && block_warps != 4)
     LMSF_REFUSE("attention_decode: blocks have 2 or 4 warps, not %d", block_warps);
@@ -701,10 +709,12 @@ static int decode_launch(lmsf::fa::DecodeArgs& a, int gy, int grid_x, int grid_z
     deep = fit[cs][R] > 0 && clusters <= fit[cs][R];
   }
   const bool one = a.kv.v_off == 0, table = a.x.dist != nullptr;      // keys that are values; a table of distances
+  const bool cap = a.x.softcap > 0.f;
+  if (cap && (one || table)) LMSF_REFUSE("attention_decode: a cap on the scores goes with keys and values of their own and no table of distances");
   if (table && !one) deep = false;
-  DecodeKernel kernel = decode_variant(warps, deep, one, table);
+  DecodeKernel kernel = decode_variant(warps, deep, one, table, cap);
   const int smem = decode_smem_bytes(a.group, warps, deep ? kDeepStages : kStages);
-  if (const cudaError_t e = decode_allow_smem(warps, smem, deep, one, table)) return (int)e;
+  if (const cudaError_t e = decode_allow_smem(warps, smem, deep, one, table, cap)) return (int)e;
   if (!a.cluster) return launch_pdl(kernel, dim3(grid_x, (unsigned)gy, grid_z), dim3(32 * warps), smem, s, a);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(grid_x, (unsigned)gy, grid_z);
@@ -753,7 +763,8 @@ LMSF_API int lmsf_attention_decode_items(const void* q, long long q_stride, void
                                          int n_seqs_total, const int* cu_q, const int* ctx_len, float scale, int window,
                                          int n_q_heads, int head_dim, int block_warps, void* scratch, int kv_planes,
                                          int chunk, const float* r1, const float* r2, const float* sinks, int keep_first,
-                                         int sigmoid, const float* head_bias, const float* dist, int dist_n, void* stream) {
+                                         int sigmoid, const float* head_bias, const float* dist, int dist_n, float softcap,
+                                         void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (capacity <= 0) return 0;
@@ -781,7 +792,7 @@ LMSF_API int lmsf_attention_decode_items(const void* q, long long q_stride, void
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_decode: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_decode: sinks belong to a softmax, not to sigmoid weights");
   if (dist && dist_n <= 0) LMSF_REFUSE("attention_decode: a table of %d distances", dist_n);
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n, softcap > 0.f ? softcap : 0.f};
   a.rows = decode_rows(group);
   a.items = (const int4*)items;
   a.cluster = 0;
@@ -797,7 +808,7 @@ LMSF_API int lmsf_attention_decode(const void* q, long long q_stride, void* out,
                                    int n_q_heads, int head_dim, int n_splits, void* scratch, void* stream) {
   return lmsf_attention_decode_width(q, q_stride, out, out_stride, cache, page_stride, block_size, n_kv_heads, block_table,
                                      max_blocks, seq_ids, n_served, n_seqs_total, cu_q, ctx_len, scale, window, n_q_heads,
-                                     head_dim, n_splits, 0, scratch, 2, 0, nullptr, nullptr, nullptr, 0, 0, nullptr, nullptr, 0, stream);
+                                     head_dim, n_splits, 0, scratch, 2, 0, nullptr, nullptr, nullptr, 0, 0, nullptr, nullptr, 0, 0.f, stream);
 }
 
 // ------------------------------------------------------------------------------------------------

@@ -71,7 +71,19 @@ struct ScoreExtras {
   const float* head_bias;   // [n_q_heads]: a number per query head added to every scaled score
   const float* dist;        // [n_q_heads][dist_n]: the entry of the distance p - key (the last entry for every distance from
   int dist_n;               // dist_n - 1 on) is added to the scaled score
+  float softcap;            // > 0: a scaled score s becomes softcap * tanh(s / softcap) before anything else is done to it
 };
+// tanh(x) / x as a polynomial in u = x^2, the series of tanh at 0 through x^9: within 1e-8 of the quotient for |x| <= kTanhSmall
+constexpr float kTanhSmall = 0.25f;
+constexpr float kTanh3 = -1.0f / 3.0f, kTanh5 = 2.0f / 15.0f, kTanh7 = -17.0f / 315.0f, kTanh9 = 62.0f / 2835.0f;
+// tanh(x): the series near 0 (exact relative to x), else 1 - 2 / (1 + e^(2x)) on the special-function unit
+__device__ __forceinline__ float tanh_large(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x * 2.8853900817779268f)); }
+__device__ __forceinline__ float tanh_score(float x) {
+  const float u = x * x;
+  float t = x * fmaf(u, fmaf(u, fmaf(u, fmaf(u, kTanh9, kTanh7), kTanh5), kTanh3), 1.0f);
+  if (fabsf(x) > kTanhSmall) t = tanh_large(x);
+  return t;
+}
 // The key tiles that a block walks when the window's keys [lo, hi) are joined by the kept first keys [0, keep): tiles
 // 0 .. n_first - 1 and then tile_lo .. tile_hi - 1 (n_first = 0 when the window's first tile reaches the kept keys anyway).
 struct TileRange {

@@ -20,8 +20,8 @@ struct PrefillArgs {
 // One block: 64 query tokens (16 per warp) of one head.  Query i of a portion of n tokens of a request
 // that holds ctx keys after this step sits at position ctx - n + i and sees keys lo..position.
 // ONE: the cache's keys are its values; a stage is half as large and there are twice as many.  TABLE: a table of distances is
-// added to the scores.
-template <bool ONE, bool TABLE>
+// added to the scores.  CAP: scores are capped smoothly.
+template <bool ONE, bool TABLE, bool CAP>
 __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   constexpr int S = ONE ? 2 * kStages : kStages, kStageBytes = ONE ? St::kBytes / 2 : St::kBytes;
   extern __shared__ __align__(16) unsigned char smem[];
@@ -82,7 +82,8 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
   float o[HD / 8][4];
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  const float sl2 = a.scale * kLog2e;
+  const float cap_in = CAP ? a.scale / a.x.softcap : 0.f;       // as in the decode kernel
+  const float sl2 = CAP ? a.x.softcap * kLog2e : a.scale * kLog2e;
 
   for (int i = 0; i < n_tiles; ++i) {
     cp_async_wait<S - 2>();
@@ -121,6 +122,7 @@ __global__ void __launch_bounds__(kThreads) prefill_kernel(PrefillArgs a) {
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + j * 8 + t4 * 2 + (e & 1), h = e >> 1;
         const bool ok = key <= pos[h] && (key >= row_lo[h] || key < keep);
+        if (CAP) s[j][e] = tanh_score(s[j][e] * cap_in);
         float v = ok ? fmaf(s[j][e], sl2, hb2) : -INFINITY;
         if (biased && ok) v -= log_distance_bias2f(r1, r2, dist0[h] - (float)(j * 8 + (e & 1)));
         if (TABLE && ok) v += table_bias2(dist_row, a.x.dist_n, pos[h] - key);
@@ -198,7 +200,7 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
                                     int n_tiles, const int* cu_q, const int* ctx_len, float scale, int window,
                                     int n_q_heads, int head_dim, int kv_planes, int chunk, const float* r1,
                                     const float* r2, const float* sinks, int keep_first, int sigmoid,
-                                    const float* head_bias, const float* dist, int dist_n, void* stream) {
+                                    const float* head_bias, const float* dist, int dist_n, float softcap, void* stream) {
   using namespace lmsf;
   using namespace lmsf::fa;
   if (n_tiles <= 0) return 0;
@@ -217,17 +219,20 @@ LMSF_API int lmsf_attention_prefill(const void* q, long long q_stride, void* out
   if ((r1 == nullptr) != (r2 == nullptr) || chunk < 0) LMSF_REFUSE("attention_prefill: the distance bias takes both constants; chunk >= 0");
   if (sigmoid && sinks) LMSF_REFUSE("attention_prefill: sinks belong to a softmax, not to sigmoid weights");
   if (dist && dist_n <= 0) LMSF_REFUSE("attention_prefill: a table of %d distances", dist_n);
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n, softcap > 0.f ? softcap : 0.f};
   const int smem = kStages * St::kBytes;
   const bool one = kv_planes == 1;
-  const bool table = dist != nullptr;
-  void (*kernel)(PrefillArgs) = table ? (one ? prefill_kernel<true, true> : prefill_kernel<false, true>)
-                                      : (one ? prefill_kernel<true, false> : prefill_kernel<false, false>);
-  static bool configured[2][2] = {{false, false}, {false, false}};
-  if (!configured[table][one]) {
+  const bool table = dist != nullptr, cap = softcap > 0.f;
+  if (cap && (one || table)) LMSF_REFUSE("attention_prefill: a cap on the scores goes with keys and values of their own and no table of distances");
+  void (*kernel)(PrefillArgs) = cap ? prefill_kernel<false, false, true>
+                                : table ? (one ? prefill_kernel<true, true, false> : prefill_kernel<false, true, false>)
+                                        : (one ? prefill_kernel<true, false, false> : prefill_kernel<false, false, false>);
+  static bool configured[5] = {false, false, false, false, false};
+  bool& ready = configured[cap ? 4 : 2 * table + one];
+  if (!ready) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    configured[table][one] = true;
+    ready = true;
   }
   kernel<<<dim3(n_q_heads, n_tiles), kThreads, smem, (cudaStream_t)stream>>>(a);
   return LMSF_LAUNCH_STATUS();

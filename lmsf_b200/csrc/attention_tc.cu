@@ -119,6 +119,11 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
   return d;
 }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -228,8 +233,9 @@ struct Unit {
 
 // kSig: sigmoid weights (a second build of the softmax warps' loop, so that the softmax form carries no test of it).  kKeep: a
 // window that keeps the request's first keys (a list of tiles with a gap); without it every count of kept tiles is a constant 0
-// and the kernel is the one it was before it learnt of them.  Built: plain, kKeep, and kSig with kKeep.
-template <bool kLeft, bool kSig, bool kKeep>
+// and the kernel is the one it was before it learnt of them.  kCap: scores are capped smoothly.  Built: plain, kKeep, kSig with
+// kKeep, and kCap.
+template <bool kLeft, bool kSig, bool kKeep, bool kCap = false>
 __global__ void __launch_bounds__(kThreadsTotal, 1) prefill_tc_kernel(const Args a, const __grid_constant__ CUtensorMap kv_map,
                                                                       const __grid_constant__ CUtensorMap q_map) {
   extern __shared__ unsigned char smem_raw[];
@@ -608,6 +614,35 @@ __global__ void __launch_bounds__(kThreadsTotal, 1) prefill_tc_kernel(const Args
 #pragma unroll
         for (int c0 = 0; c0 < BN; c0 += 32) tmem_ld32_issue(t_s + c0, sc + c0);
         tmem_wait_ld();
+        if constexpr (kCap) {
+          // softcap * tanh(s * scale / softcap) in the raw scores' units is s * (tanh(x) / x) with x = s * scale / softcap: the
+          // quotient is a polynomial in x^2 where every score of the warp's rows is small (the usual case: no special function),
+          // else tanh itself is computed
+          const float k = a.scale / a.x.softcap, k2 = k * k;
+          float big0 = fmax3(fabsf(sc[0]), fabsf(sc[1]), fabsf(sc[2])), big1 = fmaxf(fabsf(sc[3]), fabsf(sc[4]));
+          big1 = fmaxf(big1, fabsf(sc[BN - 1]));
+#pragma unroll
+          for (int i = 5; i + 3 < BN; i += 4) {
+            big0 = fmax3(big0, fabsf(sc[i]), fabsf(sc[i + 1]));
+            big1 = fmax3(big1, fabsf(sc[i + 2]), fabsf(sc[i + 3]));
+          }
+          big0 = fmax3(big0, fabsf(sc[BN - 3]), fabsf(sc[BN - 2]));
+          if (__any_sync(0xffffffffu, fmaxf(big0, big1) * fabsf(k) > kTanhSmall)) {
+            const float inv_k = a.x.softcap / a.scale;
+#pragma unroll
+            for (int i = 0; i < BN; ++i) sc[i] = tanh_score(sc[i] * k) * inv_k;
+          } else {
+            const uint64_t kk = pk2(k2, k2), c9 = pk2(kTanh9, kTanh9), c7 = pk2(kTanh7, kTanh7), c5 = pk2(kTanh5, kTanh5),
+                           c3 = pk2(kTanh3, kTanh3), one = pk2(1.f, 1.f);
+#pragma unroll
+            for (int i = 0; i < BN; i += 2) {
+              const uint64_t s2 = pk2(sc[i], sc[i + 1]);
+              const uint64_t u = mul2(mul2(s2, s2), kk);
+              const uint64_t p = fma2(u, fma2(u, fma2(u, fma2(u, c9, c7), c5), c3), one);
+              upk2(mul2(s2, p), sc[i], sc[i + 1]);
+            }
+          }
+        }
         if (a.x.r1 != nullptr || a.x.dist != nullptr) {
           // The bias is taken off the raw scores, in their own units (the scale is folded in below, with the maximum).
           // It depends on the distance alone, and the 32 rows of a warp meet the tile's 128 keys at 159 distances: the
@@ -805,7 +840,7 @@ LMSF_API int lmsf_attention_prefill_tc(const void* q, long long q_stride, long l
                                        int n_tiles, const int* cu_q, const int* ctx_len, float scale, int window,
                                        int n_q_heads, int head_dim, int* error_flag, int kv_planes, int chunk,
                                        const float* r1, const float* r2, const float* sinks, int keep_first, int sigmoid,
-                                       const float* head_bias, const float* dist, int dist_n, void* stream) {
+                                       const float* head_bias, const float* dist, int dist_n, float softcap, void* stream) {
   using namespace lmsf;
   using namespace lmsf::tc;
   if (n_tiles <= 0) return 0;
@@ -831,7 +866,7 @@ LMSF_API int lmsf_attention_prefill_tc(const void* q, long long q_stride, long l
   if (!sigmoid && head_bias) LMSF_REFUSE("attention_prefill_tc: a bias per head is taken with sigmoid weights only");
   if (dist && (dist_n <= 0 || !(scale > 0.f) || r1))
     LMSF_REFUSE("attention_prefill_tc: a table of distances has entries, a positive scale and no other distance bias beside it");
-  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n};
+  a.x = ScoreExtras{chunk, r1, r2, sinks, (window > 0 && keep_first > 0) ? keep_first : 0, sigmoid ? 1 : 0, head_bias, dist, dist_n, softcap > 0.f ? softcap : 0.f};
   // pages of 8 keys and more come by tensor-map copies (a box of rows_box keys starts on a 1024-byte
   // boundary of the swizzled tile); smaller pages by cp.async
   a.rows_box = block_size < BN ? block_size : BN;
@@ -863,12 +898,16 @@ LMSF_API int lmsf_attention_prefill_tc(const void* q, long long q_stride, long l
     LMSF_REFUSE("attention_prefill_tc: with an odd number of query heads per kv head a launch takes %d query tiles at most, not %d",
                 kMaxLeadTiles, n_tiles);
   const bool sig = a.x.sigmoid != 0;
-  const int form = sig ? 2 : (a.x.keep_first > 0 ? 1 : 0);
+  const bool cap = a.x.softcap > 0.f;
+  if (cap && (sig || a.x.keep_first > 0 || !(scale > 0.f)))
+    LMSF_REFUSE("attention_prefill_tc: a cap on the scores goes with a softmax, a positive scale and no kept first keys");
+  const int form = cap ? 3 : sig ? 2 : (a.x.keep_first > 0 ? 1 : 0);
   void (*kernel)(const Args, const CUtensorMap, const CUtensorMap) =
-      form == 2 ? (left ? prefill_tc_kernel<true, true, true> : prefill_tc_kernel<false, true, true>)
+      form == 3 ? (left ? prefill_tc_kernel<true, false, false, true> : prefill_tc_kernel<false, false, false, true>)
+      : form == 2 ? (left ? prefill_tc_kernel<true, true, true> : prefill_tc_kernel<false, true, true>)
       : form == 1 ? (left ? prefill_tc_kernel<true, false, true> : prefill_tc_kernel<false, false, true>)
                   : (left ? prefill_tc_kernel<true, false, false> : prefill_tc_kernel<false, false, false>);
-  static bool configured[3][2] = {{false, false}, {false, false}, {false, false}};
+  static bool configured[4][2] = {{false, false}, {false, false}, {false, false}, {false, false}};
   if (!configured[form][left]) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
     if (e != cudaSuccess) return (int)e;

@@ -3,7 +3,8 @@
 // them: the short causal convolution over time with its carried inputs, and the norm over groups of columns with a gate.
 //
 //   causal_conv   y[t, c] = act(b[c] + sum_j w[c, j] * x[t - (taps - 1) + j, c]); inputs before a portion's first token
-//                 come from the request's state slot ([taps - 1, channels] float32), which is rolled on afterwards
+//                 come from the request's state slot ([taps - 1, channels] float32), which is rolled on afterwards; act is
+//                 silu, nothing, or the sum with the input itself (x[t, c] + ...)
 //   gated_scan    per request, head and token, in this order:
 //                   dt = softplus(raw_dt + dt_bias[h]);  a = exp(-exp(a_log[h]) * dt)
 //                   plain rule:  S <- a S + (dt k) v^T                      (k_times_dt; the write is k v^T without it)
@@ -32,12 +33,17 @@ __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log
 
 constexpr int kConvChannels = 64;    // channels per block (threadIdx.x)
 constexpr int kConvChunk = 256;      // tokens per block along gridDim.z
-constexpr int kMaxTaps = 8;
+constexpr int kMaxTaps = 32;
+enum { kConvPlain = 0, kConvSilu = 1, kConvAddInput = 2 };
+__device__ __forceinline__ float conv_end(float acc, float x, int act) {
+  return act == kConvSilu ? silu_f(acc) : (act == kConvAddInput ? x + acc : acc);
+}
 
+// MAXT: taps that a build holds in registers.
 // grid (channel tiles, requests, token chunks); block (64, lanes): lanes of tokens side by side.
 // Only the block of a request's first chunk reads its state, and only that block writes it (after its outputs):
 // later chunks start at least kConvChunk >= taps - 1 tokens into the portion.
-template <typename T>
+template <typename T, int MAXT>
 __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, const T* __restrict__ x, long long x_stride,
                                    const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                                    long long slot_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slot,
@@ -50,21 +56,22 @@ __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, co
   const int hi = min(n, lo + kConvChunk);
   float* st = state + (size_t)state_slot[s] * slot_stride;      // [taps - 1][C]
   if (c < C) {
-    float wr[kMaxTaps];
+    float wr[MAXT];
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j) wr[j] = j < taps ? w[(size_t)c * taps + j] : 0.f;
+    for (int j = 0; j < MAXT; ++j) wr[j] = j < taps ? w[(size_t)c * taps + j] : 0.f;
     const float b = bias ? bias[c] : 0.f;
     for (int t = lo + threadIdx.y; t < hi; t += blockDim.y) {
-      float acc = b;
+      float acc = b, last = 0.f;
 #pragma unroll
-      for (int j = 0; j < kMaxTaps; ++j) {
+      for (int j = 0; j < MAXT; ++j) {
         if (j < taps) {
           const int u = t - (taps - 1) + j;                     // place in the portion; negative: before it
           const float v = u >= 0 ? to_f32(x[(size_t)(t0 + u) * x_stride + c]) : st[(size_t)(taps - 1 + u) * C + c];
           acc = fmaf(wr[j], v, acc);
+          last = v;                                             // the last tap's input is the token's own
         }
       }
-      out[(size_t)(t0 + t) * out_stride + c] = from_f32<T>(act ? silu_f(acc) : acc);
+      out[(size_t)(t0 + t) * out_stride + c] = from_f32<T>(conv_end(acc, last, act));
     }
   }
   if (blockIdx.z != 0) return;
@@ -147,7 +154,7 @@ __global__ void __launch_bounds__(kConvVecThreads) causal_conv_vec_kernel(
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) a = fmaf(wr[j][e], win[j][e], a);
       a = fmaf(wr[TAPS - 1][e], cur[e], a);
-      acc[e] = act ? silu_f(a) : a;
+      acc[e] = conv_end(a, cur[e], act);
     }
     conv_store<T, VEC>(out + (size_t)(t0 + t) * out_stride + c, acc);
 #pragma unroll
@@ -458,31 +465,32 @@ __global__ void __launch_bounds__(BLOCK ? 256 : 128) grouped_gated_norm_reg_kern
 }  // namespace lmsf
 
 // x: [n, C] rows of `dtype` with x_stride elements between tokens; out likewise; w: float32 [C, taps]; bias: float32 [C] or
-// null; state: float32, the [taps - 1, C] block of slot s starts at state + s * slot_stride.  act: 0 none, 1 silu.
+// null; state: float32, the [taps - 1, C] block of slot s starts at state + s * slot_stride.  act: 0 none, 1 silu, 2 the input added.
 // max_q: the longest portion of the launch (the host's copy; sizes the grid only).
 LMSF_API int lmsf_causal_conv(void* out, long long out_stride, const void* x, long long x_stride, const float* w,
                               const float* bias, float* state, long long slot_stride, const int* cu_q, const int* state_slot,
                               int n_seqs, int max_q, int C, int taps, int act, int dtype, void* stream) {
   using namespace lmsf;
   if (n_seqs <= 0 || max_q <= 0) return 0;
+  if (act < kConvPlain || act > kConvAddInput) LMSF_REFUSE("causal_conv: unknown ending %d", act);
   if (C <= 0 || taps < 1 || taps > kMaxTaps) LMSF_REFUSE("causal_conv: %d channels, %d taps (1 to %d taps)", C, taps, kMaxTaps);
   if (n_seqs > 65535) LMSF_REFUSE("causal_conv: more than 65535 requests in one launch");
   cudaStream_t s = (cudaStream_t)stream;
   if (ceil_div(max_q, kConvVecChunk) > 65535) LMSF_REFUSE("causal_conv: a portion of %d tokens is too long for one launch", max_q);
   // 16-byte accesses where the rows allow them (the state's rows are then 16-byte aligned too)
   const int vec = dtype == LMSF_F32 ? 4 : 8;
-  if ((dtype == LMSF_F32 || dtype == LMSF_BF16) && C % vec == 0 && out_stride % vec == 0 && x_stride % vec == 0 &&
+  if ((dtype == LMSF_F32 || dtype == LMSF_BF16) && taps <= 8 && C % vec == 0 && out_stride % vec == 0 && x_stride % vec == 0 &&
       ((uintptr_t)out | (uintptr_t)x) % 16 == 0) {
     if (dtype == LMSF_F32) return launch_conv_vec<float, 4>(out, out_stride, x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, n_seqs, max_q, C, taps, act, s);
     return launch_conv_vec<bf16, 8>(out, out_stride, x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, n_seqs, max_q, C, taps, act, s);
   }
   dim3 grid(ceil_div(C, kConvChannels), n_seqs, ceil_div(max_q, kConvChunk));
   dim3 block(kConvChannels, max_q >= 4 ? 4 : (max_q >= 2 ? 2 : 1));
-  if (dtype == LMSF_F32)
-    causal_conv_kernel<float><<<grid, block, 0, s>>>((float*)out, out_stride, (const float*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, taps, act);
-  else if (dtype == LMSF_BF16)
-    causal_conv_kernel<bf16><<<grid, block, 0, s>>>((bf16*)out, out_stride, (const bf16*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, taps, act);
+#define LMSF_GO(T, M) causal_conv_kernel<T, M><<<grid, block, 0, s>>>((T*)out, out_stride, (const T*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, taps, act)
+  if (dtype == LMSF_F32) { if (taps <= 8) LMSF_GO(float, 8); else LMSF_GO(float, kMaxTaps); }
+  else if (dtype == LMSF_BF16) { if (taps <= 8) LMSF_GO(bf16, 8); else LMSF_GO(bf16, kMaxTaps); }
   else LMSF_REFUSE("causal_conv: unknown dtype code %d", dtype);
+#undef LMSF_GO
   return LMSF_LAUNCH_STATUS();
 }
 

@@ -670,14 +670,15 @@ def _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, wha
 
 
 
-def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=False, head_bias=None, dist=None):
-    """(chunk, r1, r2, sinks, keep_first, sigmoid, head_bias, dist, its entries) as the tensor-core attention kernels take them: what a design
+def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=False, head_bias=None, dist=None, softcap=0.0):
+    """(chunk, r1, r2, sinks, keep_first, sigmoid, head_bias, dist, its entries, softcap) as the tensor-core attention kernels take them: what a design
     adds to the causal softmax.  chunk > 0: a query at position p sees the keys p - p % chunk .. p only.  log_bias (r1, r2),
     float32 [n_q_heads] each: r1 * log(1 + r2 * distance) is taken off the scaled scores.  sinks, float32 [n_q_heads]:
     exp(sink) is one more term of the softmax's denominator.  keep_first (with a window): the request's first keys stay
     visible behind it.  sigmoid: a visible key's weight is sigmoid(score), not normalised.  head_bias, float32 [n_q_heads]:
     added to the scaled scores.  dist, float32 [n_q_heads, entries]: the entry of the distance (the last one for every larger
-    distance) is added to the scaled score."""
+    distance) is added to the scaled score.  softcap > 0: a scaled score s becomes softcap * tanh(s / softcap) before anything
+    is added to it (keys and values of their own and no table of distances)."""
     _per_head(head_bias, n_q_heads, "the bias per head")
     r1, r2 = log_bias if log_bias is not None else (None, None)
     _per_head(r1, n_q_heads, "the logarithmic bias")
@@ -686,7 +687,7 @@ def _score_extras(n_q_heads: int, chunk, log_bias, sinks, keep_first=0, sigmoid=
     if chunk is not None and int(chunk) < 0:
         raise KernelError(f"attention: a chunk of {chunk} positions")
     return int(chunk or 0), _ptr(r1), _ptr(r2), _ptr(sinks), int(keep_first or 0), 1 if sigmoid else 0, _ptr(head_bias), \
-        *_dist_args(dist, n_q_heads)
+        *_dist_args(dist, n_q_heads), float(softcap or 0.0)
 
 
 _DECODE_WIDTHS = {}
@@ -782,7 +783,8 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
                      ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int,
                      head_dim: int, n_splits: int, scratch: Optional[torch.Tensor], warps: int = 0, kv_planes: int = 2,
                      chunk: int = 0, log_bias=None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                     sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
+                     sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                     softcap: float = 0.0):
     """Attention of requests that bring ONE query token each (row cu_q[s] of q), over their ctx_len[s] keys
     in pages.  seq_ids: int32 [n_served] rows of the block table that are served (None: all, in order).
     scratch: float32, at least attention_decode_scratch_floats(...) values when n_splits > 1, all zero when it is
@@ -791,7 +793,7 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
     kv_planes 1: the cache holds one vector per token and kv head that is key and value at once.
     chunk, log_bias, sinks: see _score_extras."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_decode", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist, softcap)
     n_total = block_table.shape[0]
     need = attention_decode_scratch_floats(n_total, n_q_heads, n_splits, head_dim)
     if need and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need):
@@ -802,7 +804,7 @@ def attention_decode(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, bl
     f = _func("attention_mma.cu", "lmsf_attention_decode_width",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p,
-               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
+               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_ids, "seq_ids"), n_served, n_total,
            _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale), int(window or 0), n_q_heads, head_dim,
@@ -841,11 +843,12 @@ def attention_decode_items(out: torch.Tensor, q: torch.Tensor, cache: torch.Tens
                            scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int, warps: int,
                            scratch: torch.Tensor, kv_planes: int = 2, chunk: int = 0, log_bias=None,
                            sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                           sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
+                           sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                           softcap: float = 0.0):
     """attention_decode with splits per request, over a list made by decode_build_items.  scratch: float32, at
     least attention_decode_items_scratch_floats(capacity, ...) values, zero when first used."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_decode_items", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist, softcap)
     need = attention_decode_items_scratch_floats(items.shape[0], n_q_heads, head_dim)
     if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
         raise KernelError(f"attention_decode_items: a list of {items.shape[0]} entries needs {need} float32 values of scratch")
@@ -853,7 +856,7 @@ def attention_decode_items(out: torch.Tensor, q: torch.Tensor, cache: torch.Tens
     f = _func("attention_mma.cu", "lmsf_attention_decode_items",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int, c_void_p, c_int,
-               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
+               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _ptr(items), items.shape[0], block_table.shape[0],
            _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale), int(window or 0), n_q_heads, head_dim, int(warps),
@@ -865,16 +868,17 @@ def attention_prefill(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, b
                       block_size: int, tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, cu_q: torch.Tensor,
                       ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int,
                       kv_planes: int = 2, chunk: int = 0, log_bias=None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                      sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
+                      sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                      softcap: float = 0.0):
     """Attention of prompt portions.  Tile i covers the query tokens tile_q0[i] .. tile_q0[i] + 63 (counted
     inside the portion) of request tile_seq[i]."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_prefill", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist, softcap)
     d = _mma_defines(head_dim)
     f = _func("attention_mma.cu", "lmsf_attention_prefill",
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_int,
                c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int,
-               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
+               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), block_size, n_kv_heads,
            _i32(block_table, "block_table"), block_table.shape[1], _i32(tile_seq, "tile_seq"),
            _i32(tile_q0, "tile_q0"), n_tiles, _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale),
@@ -897,16 +901,17 @@ def attention_prefill_tc(out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor
                          ctx_len: torch.Tensor, scale: float, window: int, n_q_heads: int, n_kv_heads: int, head_dim: int,
                          error_flag: Optional[torch.Tensor] = None, kv_planes: int = 2, chunk: int = 0, log_bias=None,
                          sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                         sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None):
+                         sigmoid: bool = False, head_bias: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                         softcap: float = 0.0):
     """Attention of prompt portions on tcgen05 tensor cores (head size 64 or 128).  Tile i covers the query
     tokens tile_q0[i] .. tile_q0[i] + 127 (counted inside the portion) of request tile_seq[i]."""
     _check_paged(q, out, cache, n_q_heads, n_kv_heads, head_dim, block_size, "attention_prefill_tc", kv_planes)
-    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist)
+    extras = _score_extras(n_q_heads, chunk, log_bias, sinks, keep_first, sigmoid, head_bias, dist, softcap)
     d = _mma_defines(head_dim)[:1]
     f = _func("attention_tc.cu", "lmsf_attention_prefill_tc",
               [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_int, c_int,
                c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p,
-               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], d)
+               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p], d)
     rc = f(_ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), cache.shape[0], block_size,
            n_kv_heads, _i32(block_table, "block_table"), block_table.shape[1], _i32(tile_seq, "tile_seq"),
            _i32(tile_q0, "tile_q0"), n_tiles, _i32(cu_q, "cu_q"), _i32(ctx_len, "ctx_len"), float(scale),
@@ -1012,6 +1017,77 @@ def token_shift(out: torch.Tensor, h: torch.Tensor, mix: torch.Tensor, state: to
     rc = f(_ptr(out), _ptr(h), _f32vec(mix, hidden, "mix"), _ptr(state), _i32(positions, "positions"),
            _i32(token_seq, "token_seq"), _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), n, hidden, dtype_code(h.dtype), _stream())
     _check(rc, "stream_norm.cu", "lmsf_stream_norm")
+
+
+def stream_layer(res: torch.Tensor, y: Optional[torch.Tensor] = None, pair=None, w_post: Optional[torch.Tensor] = None,
+                 eps_post: float = 0.0, post_centred: bool = False, vec: Optional[torch.Tensor] = None,
+                 h: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0,
+                 next_centred: bool = False, filt=None):
+    """What lies between two branches, for norms that may take the mean off: res += N_post(b); res += vec; h = N_next(res), and
+    behind it, for rows that are single tokens, a short filter over time, h + sum_j f[:, j] * h of the tokens before and its own.
+    N(x) = (x - mean) / sqrt(variance + eps) * w where centred, else x / rms(x) * w.  b = y, or with `pair` (y2, p1, p2, eps,
+    factor) b = factor * (y / rms(y) * p1 + y2 / rms(y2) * p2).  `filt` (f float32 [hidden, taps], state float32 [slots,
+    (taps - 1) * hidden], state_slot int32 [n]): row i is the token of slot state_slot[i], whose inputs are rolled on.
+    res: float32 [n, hidden]; y, y2, h: contiguous [n, hidden] of one activation type; vectors float32 [hidden]."""
+    n, hidden = res.shape
+    if res.dtype != torch.float32 or not res.is_contiguous():
+        raise KernelError("stream_layer: the residual stream must be contiguous float32")
+    y2, p1, p2, pair_eps, factor = pair if pair is not None else (None, None, None, 0.0, 0.0)
+    given = [t for t in (y, y2, h) if t is not None]
+    for t in given:
+        if t.shape != res.shape or not t.is_contiguous() or t.dtype != given[0].dtype:
+            raise KernelError("stream_layer: branches and output must be contiguous, of the stream's shape and of one activation type")
+    f, taps, state, slots = None, 0, None, None
+    if filt is not None:
+        f, state, slots = filt
+        taps = f.shape[1]
+        if f.dtype != torch.float32 or f.shape[0] != hidden or not f.is_contiguous() or state.dtype != torch.float32 or \
+                not state.is_contiguous() or state.dim() != 2 or state.shape[1] < (taps - 1) * hidden or slots.numel() != n:
+            raise KernelError("stream_layer: the filter is float32 [hidden, taps], its state float32 [slots, (taps - 1) * hidden], one slot a row")
+    fn = _func("layer_norm.cu", "lmsf_stream_layer",
+               [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_float, c_int, c_void_p, c_void_p,
+                c_void_p, c_float, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p])
+    rc = fn(_ptr(res), _ptr(y), _ptr(y2), _f32vec(p1, hidden, "p1"), _f32vec(p2, hidden, "p2"), float(pair_eps), float(factor),
+            _f32vec(w_post, hidden, "w_post"), float(eps_post), int(post_centred), _f32vec(vec, hidden, "vec"), _ptr(h),
+            _f32vec(w_next, hidden, "w_next"), float(eps_next), int(next_centred), _ptr(f), taps, _ptr(state),
+            state.stride(0) if state is not None else 0, _i32(slots, "state_slot"), n, hidden,
+            dtype_code(given[0].dtype) if given else F32, _stream())
+    _check(rc, "layer_norm.cu", "lmsf_layer_norm")
+
+
+def conv_rope_cache_write(q: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, state_offset: int,
+                          cu_q: torch.Tensor, state_slot: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor,
+                          block_size: int, cache: torch.Tensor, inv_freq: Optional[torch.Tensor], rot_dim: int, mult: float,
+                          n_q_heads: int, n_kv_heads: int, head_dim: int, n_seqs: int, max_q: int,
+                          error_flag: Optional[torch.Tensor] = None):
+    """Queries and keys through a short causal filter over time: x [n, (n_q_heads + n_kv_heads) * head_dim] (a view) -> q [n,
+    n_q_heads * head_dim] filtered and turned; the keys filtered and turned into plane 0 of their page, filtered alone into plane
+    1 (the values).  w: float32 [taps, channels]; the taps - 1 inputs before a portion are state[slot, state_offset:][: (taps - 1)
+    * channels] (float32), rolled on.  Pairs (i, i + rot_dim / 2) turn by position * inv_freq[i], cos and sin times mult."""
+    n, C = x.shape
+    taps = w.shape[0]
+    if C != (n_q_heads + n_kv_heads) * head_dim:
+        raise KernelError("conv_rope: x must hold the query heads and the key heads side by side")
+    _rows(x, C, "conv_rope: x")
+    _rows(q, n_q_heads * head_dim, "conv_rope: q", x.dtype)
+    if w.dtype != torch.float32 or w.shape != (taps, C) or not w.is_contiguous():
+        raise KernelError("conv_rope: w must be contiguous float32 [taps, channels]")
+    if state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state_offset < 0 or \
+            state_offset + (taps - 1) * C > state.shape[1]:
+        raise KernelError("conv_rope: the state must be contiguous float32 [slots, size] with room for [taps - 1, channels]")
+    if cache.dtype != x.dtype or not cache.is_contiguous() or tuple(cache.shape[1:]) != (2, n_kv_heads, block_size, head_dim):
+        raise KernelError(f"conv_rope: cache of shape {tuple(cache.shape)} does not match [pages, 2, {n_kv_heads}, {block_size}, {head_dim}] of {x.dtype}")
+    if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dim // 2):
+        raise KernelError("conv_rope: inv_freq must hold rot_dim / 2 float32 values")
+    f = _func("conv_rope.cu", "lmsf_conv_rope_cache",
+              [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
+               c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
+               c_void_p, c_void_p])
+    rc = f(_ptr(x), x.stride(0), _ptr(q), q.stride(0), _ptr(w), taps, _ptr(state) + 4 * state_offset, state.stride(0),
+           _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), _i32(positions, "positions"), _i32(block_table, "block_table"),
+           block_table.shape[1], block_size, _ptr(cache), cache.stride(0), _ptr(inv_freq), rot_dim, float(mult), n_q_heads, n_kv_heads,
+           head_dim, n_seqs, int(max_q), dtype_code(x.dtype), _i32(error_flag, "error_flag"), _stream())
+    _check(rc, "conv_rope.cu", "lmsf_conv_rope")
 
 
 def stream_concat(out: torch.Tensor, a: torch.Tensor, b: torch.Tensor):
@@ -1123,7 +1199,8 @@ def gated_norm(out: torch.Tensor, x: torch.Tensor, gate: torch.Tensor, w: torch.
 
 # ----------------------------------------------------------------------------- recurrent mixers with a state matrix per head
 
-CONV_MAX_TAPS = 8
+CONV_MAX_TAPS = 32
+CONV_ACTS = {None: 0, "none": 0, "silu": 1, "add_input": 2}
 SCAN_MAX_DK = 256
 
 
@@ -1136,7 +1213,8 @@ def causal_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Optio
                 state_offset: int, cu_q: torch.Tensor, state_slot: torch.Tensor, n_seqs: int, max_q: int, act: str = "silu"):
     """out[t, c] = act(bias[c] + sum_j w[c, j] x[t - (taps - 1) + j, c]) per request (tokens cu_q[s]..cu_q[s + 1]); the
     inputs before a portion come from state[slot, state_offset : state_offset + (taps - 1) * C] ([taps - 1, C], float32),
-    which then takes the portion's last inputs.  x, out: [n, C] views; w: float32 [C, taps]; state: float32 [slots, size]."""
+    which then takes the portion's last inputs.  act "add_input": the input itself is added, x[t, c] + sum.
+    x, out: [n, C] views; w: float32 [C, taps]; state: float32 [slots, size]."""
     n, C = x.shape
     taps = w.shape[1]
     _rows(x, C, "causal_conv: x")
@@ -1151,7 +1229,7 @@ def causal_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Optio
                c_int, c_int, c_int, c_int, c_int, c_void_p])
     rc = f(_ptr(out), out.stride(0), _ptr(x), x.stride(0), _ptr(w), _f32vec(bias, C, "bias"),
            state.data_ptr() + 4 * state_offset, state.stride(0), _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), n_seqs,
-           int(max_q), C, taps, {"none": 0, None: 0, "silu": 1}[act], dtype_code(x.dtype), _stream())
+           int(max_q), C, taps, CONV_ACTS[act], dtype_code(x.dtype), _stream())
     _check(rc, "recurrent.cu", "lmsf_recurrent")
 
 

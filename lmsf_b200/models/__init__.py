@@ -1,2 +1,2 @@
 """Architectures.  Importing this package registers them."""
-from . import bedenex, fivedra, llama, redarax, vufolorn, zonidra  # noqa: F401
+from . import bedenex, dizepel, fivedra, llama, redarax, vufolorn, zonidra  # noqa: F401

@@ -17,7 +17,7 @@ from typing import Dict, Optional
 import torch
 
 from .. import kernels
-from .base import (KVCacheSpec, LayerCache, Mixer, NormAfter, PositionEncoding, Prenormed, StepContext, WeightSpec,
+from .base import (KVCacheSpec, LayerCache, Mixer, NormAfter, PositionEncoding, Prenormed, StateSpec, StepContext, WeightSpec,
                    register_part)
 from . import linear
 from .linear import matmul_tn, matmul_tn_residual
@@ -42,7 +42,7 @@ class PagedAttention(Mixer):
                  head_gate: bool = False, keep_first: int = 0, score_weights: str = "softmax", head_bias: bool = False,
                  value_gate: bool = False, own_kv: bool = True, cache_window="own",
                  cache_keep_first: Optional[int] = None, values_are_keys: bool = False, unit_sink: bool = False,
-                 out_bias: Optional[bool] = None):
+                 out_bias: Optional[bool] = None, qk_filter: int = 0, learned_sink: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot be grouped over {num_kv_heads} kv heads")
         # head_dim is the stored size of a query or key head, value_dim that of a value head (default: the same).  The
@@ -94,7 +94,22 @@ class PagedAttention(Mixer):
         # values_are_keys: a token's value is its key (as it stands in the cache); there is no value projection and the cache
         # holds one vector per token and kv head.  unit_sink: one is added to the softmax's denominator (a sink of score 0)
         self.values_are_keys, self.unit_sink = bool(values_are_keys), bool(unit_sink)
-        self.kv_planes = 1 if self.values_are_keys else 2
+        # qk_filter n: queries and keys pass a causal filter of n taps per channel over time (weight `qk_filter`) behind the
+        # projection, before they are rotated; a token's value is its key BEFORE the rotation, so the cache holds both.  The last
+        # n - 1 projected rows are the request's state.  learned_sink: exp(sink), a learned number per query head (weight `sink`),
+        # joins the softmax's denominator
+        self.qk_filter_taps, self.learned_sink = int(qk_filter or 0), bool(learned_sink)
+        if self.qk_filter_taps:
+            if not self.values_are_keys:
+                raise ValueError("queries and keys that pass a filter are built for values that are the keys")
+            if not (1 <= self.qk_filter_taps <= kernels.CONV_MAX_TAPS):
+                raise ValueError(f"a filter of {qk_filter} taps is beyond the kernel (1 to {kernels.CONV_MAX_TAPS})")
+        if self.learned_sink and (self.unit_sink or score_weights != "softmax"):
+            raise ValueError("a learned sink belongs to a softmax without another sink")
+        self.kv_planes = 1 if self.values_are_keys and not self.qk_filter_taps else 2
+        self.qk_filter: Optional[torch.Tensor] = None
+        self.sink: Optional[torch.Tensor] = None
+        self._filter32: Optional[torch.Tensor] = None
         if self.values_are_keys and (self.value_dim != self.qk_dim or qk_norm or self.head_gate or self.value_gate or not self.own_kv):
             raise ValueError("values that are the keys have the keys' size and are not built with norms, gates or another call's keys")
         if self.unit_sink and self.sigmoid_weights:
@@ -109,8 +124,7 @@ class PagedAttention(Mixer):
         self.position_encoding = position_encoding
         self.window = int(window) if window else None
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
-        # scores capped smoothly, softcap * tanh(score / softcap), before the softmax (not a Llama constant).  Only the
-        # generic kernel takes it: a part built with a cap runs on that kernel in bfloat16 too, which is right and slow
+        # scores capped smoothly, softcap * tanh(score / softcap), before the softmax (not a Llama constant)
         self.softcap = float(softcap) if softcap else 0.0
         self.q_size = num_heads * head_dim
         self.kv_size = num_kv_heads * head_dim
@@ -132,6 +146,10 @@ class PagedAttention(Mixer):
             specs["qkv_bias"] = WeightSpec([(H * dk,), (G * dk,)] + ([] if self.values_are_keys else [(G * dv,)]))
         if self.has_out_bias:
             specs["o_bias"] = WeightSpec([(D,)])
+        if self.qk_filter_taps:
+            specs["qk_filter"] = WeightSpec([(H * dk, self.qk_filter_taps), (G * dk, self.qk_filter_taps)], keep_fp32=True)
+        if self.learned_sink:
+            specs["sink"] = WeightSpec([(H,)], keep_fp32=True)
         if self.qk_norm and self.qk_norm_weights:
             specs["q_norm"] = WeightSpec([(dk,)], keep_fp32=True)
             specs["k_norm"] = WeightSpec([(dk,)], keep_fp32=True)
@@ -148,7 +166,7 @@ class PagedAttention(Mixer):
                 out[:, :size] = t
                 return out.reshape(heads * hd, *t.shape[2:])
 
-            for name in ("qkv", "qkv_bias"):
+            for name in ("qkv", "qkv_bias", "qk_filter"):
                 if name in tensors and self.values_are_keys:
                     t = tensors[name]
                     tensors[name] = torch.cat([pad_heads(t[:H * dk], H, dk), pad_heads(t[H * dk:], G, dk)], 0).contiguous()
@@ -177,6 +195,12 @@ class PagedAttention(Mixer):
         return KVCacheSpec(self.num_kv_heads, self.head_dim, self.cache_window, planes=self.kv_planes,
                            keep_first=self.cache_keep_first if self.cache_window else 0)
 
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((self.filter_state_floats(),)) if self.filter_state_floats() else None
+
+    def filter_state_floats(self) -> int:
+        return max(0, self.qk_filter_taps - 1) * (self.q_size + self.kv_size)
+
     def activation_width(self) -> int:
         # q, k, v and the attention's output; the logits of a gate per element ride in the merged product
         return 2 * self.q_size + 2 * self.kv_size + (self.num_heads * self.value_dim if self.value_gate else 0)
@@ -186,6 +210,10 @@ class PagedAttention(Mixer):
             self.position_encoding.prepare(dtype, device)
         if self.qk_norm and self.qk_norm_weights:
             self._qn32, self._kn32 = self.q_norm.float().contiguous(), self.k_norm.float().contiguous()
+        if self.qk_filter_taps:
+            self._filter32 = self.qk_filter.float().t().contiguous()            # [taps][channels]
+        if self.learned_sink:
+            self._sinks = self.sink.float().contiguous()
         if self.unit_sink:
             self._sinks = torch.zeros(self.num_heads, dtype=torch.float32, device=device)
         if self.has_head_bias:
@@ -195,8 +223,10 @@ class PagedAttention(Mixer):
             warnings.warn(f"head_dim {self.head_dim} is beyond the tensor-core attention kernels "
                           f"(up to {kernels.MMA_MAX_HEAD_DIM}); bfloat16 attention runs on the generic kernel",
                           RuntimeWarning, stacklevel=2)
-        elif dtype == torch.bfloat16 and (self.softcap or self._slopes() is not None):
-            warnings.warn("a cap on the attention scores, or a bias that is linear in the distance, is taken by the generic "
+        elif dtype == torch.bfloat16 and (self._slopes() is not None or
+                                          not cap_on_tensor_cores(self.softcap, self.scale, self.kv_planes, self._dist_table(),
+                                                                  self.keep_first if self.window else 0, self.sigmoid_weights)):
+            warnings.warn("a bias that is linear in the distance, or this part's cap on the scores, is taken by the generic "
                           "kernel only; bfloat16 attention runs on it", RuntimeWarning, stacklevel=2)
         slopes = self._slopes()
         if slopes is not None and slopes.numel() != self.num_heads:
@@ -250,7 +280,31 @@ class PagedAttention(Mixer):
                                      self.num_kv_heads, self.head_dim, ctx.error_flag)
         self.attend(ctx, out, q, cache.kv, group)
 
+    def attend_filtered(self, ctx: StepContext, p: torch.Tensor, cache: LayerCache, out: torch.Tensor, state_offset: int = 0) -> None:
+        """From the projected rows of queries and keys (a view [n, q_size + kv_size]) through the filter, the rotation and the cache
+        to the heads' outputs in `out`; the filter's carried inputs start at `state_offset` of the state slot."""
+        if not cache.owner:
+            raise ValueError("queries and keys that pass a filter are built with a cache of their own")
+        group = ctx.groups[cache.group]
+        fused = self.position_encoding.fused_rotary() if self.position_encoding is not None else None
+        if (fused is None and not self._no_rotation()) or (fused is not None and not fused[2]):
+            raise ValueError("filtered queries and keys take a rotation of halves, a bias on the scores or none")
+        inv_freq, rot_dim, _ = fused if fused is not None else (None, 0, True)
+        q = torch.empty((ctx.n_tokens, self.q_size), dtype=p.dtype, device=p.device)
+        kernels.conv_rope_cache_write(q, p, self._filter32, cache.state, state_offset, ctx.cu_q, ctx.state_slot, ctx.positions,
+                                      group.block_table, group.block_size, cache.kv, inv_freq, rot_dim,
+                                      self.position_encoding.rotary_multiplier() if fused is not None else 1.0, self.num_heads,
+                                      self.num_kv_heads, self.head_dim, ctx.n_seqs, max(ctx.max_q_len, 1), ctx.error_flag)
+        self.attend(ctx, out, q, cache.kv, group)
+
     def forward(self, ctx: StepContext, h, cache: LayerCache, then: Optional[NormAfter] = None):
+        if self.qk_filter_taps:
+            p = matmul_tn(h, self.qkv, bias=self.qkv_bias)
+            out = torch.empty((ctx.n_tokens, self.q_size), dtype=p.dtype, device=p.device)
+            self.attend_filtered(ctx, p, cache, out)
+            return self._project_out(out, then)
+        if self.position_encoding is not None and self.position_encoding.rotary_multiplier() != 1.0:
+            raise ValueError("a rotation that also stretches is built with filtered queries and keys")
         if self.values_are_keys:
             p, cached = self.project(ctx, h, self.qkv, self.qkv_bias, cache)
             out = torch.empty((ctx.n_tokens, self.q_size), dtype=p.dtype, device=p.device)
@@ -337,6 +391,11 @@ class PagedAttention(Mixer):
                      head_bias=self._hb32, sinks=self._sinks, dist=self._dist_table(), kv_planes=self.kv_planes)
 
 
+def cap_on_tensor_cores(softcap: float, scale: float, kv_planes: int = 2, dist=None, keep_first: int = 0, sigmoid: bool = False) -> bool:
+    """Whether the tensor-core kernels take a cap on the scores together with these."""
+    return not softcap or (scale > 0 and kv_planes == 2 and dist is None and not keep_first and not sigmoid)
+
+
 def paged_attend(ctx: StepContext, out: torch.Tensor, q: torch.Tensor, kv: torch.Tensor, group, *, num_heads: int,
                  num_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None, softcap: float = 0.0,
                  slopes: Optional[torch.Tensor] = None, kv_planes: int = 2, chunk: Optional[int] = None,
@@ -351,11 +410,12 @@ def paged_attend(ctx: StepContext, out: torch.Tensor, q: torch.Tensor, kv: torch
     the softmax's denominator (all three: every kernel); gate [n, heads]: the output of head h is multiplied by
     sigmoid(gate[:, h]) (the generic kernel itself, a small kernel after the fast ones).  keep_first: with a window, the
     request's first keys stay visible behind it; sigmoid: a key's weight is sigmoid(score), not normalised; head_bias [heads]:
-    added to the scaled scores; dist [heads, entries]: a number per (head, distance) added to them."""
-    if kernels.mma_attention_supported(q.dtype, head_dim) and not softcap and slopes is None and \
-            not ctx.extras.get("force_generic_attention"):
+    added to the scaled scores; dist [heads, entries]: a number per (head, distance) added to them; softcap: a scaled score s
+    becomes softcap * tanh(s / softcap) first (`cap_on_tensor_cores`)."""
+    if kernels.mma_attention_supported(q.dtype, head_dim) and slopes is None and \
+            cap_on_tensor_cores(softcap, scale, kv_planes, dist, keep_first if window else 0, sigmoid) and not ctx.extras.get("force_generic_attention"):
         extras = dict(chunk=chunk or 0, log_bias=log_bias, sinks=sinks, keep_first=keep_first if window else 0,
-                      sigmoid=sigmoid, head_bias=head_bias, dist=dist)
+                      sigmoid=sigmoid, head_bias=head_bias, dist=dist, softcap=softcap)
         if ctx.n_decode_seqs:
             max_ctx = ctx.extras.get("decode_max_ctx")
             if max_ctx is None:

@@ -205,6 +205,7 @@ class Norm(Part):
     # True when the norm is a factor per row times a weight per column, so that the products around it can share its
     # work (`NormAfter`, `Prenormed`); such a norm has `weight`, `eps`, `hidden_size` and `finish`.
     splittable = False
+    centred = False         # the mean is taken off before the division (layer norm)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
@@ -243,10 +244,24 @@ class Prenormed:
 class Normed:
     """The residual stream `res` holds every branch so far and `h` is already `norm` of it: what a block returns as
     x when it has applied the next block's first norm itself (or None as x: nothing is pending, no norm applied).
-    `norm` None: the next block's branches read the stream itself, and `h` is the stream in the activation type."""
+    `norm` None: the next block's branches read the stream itself, and `h` is the stream in the activation type.
+    `shifted`: h has passed the next block's first `Shift` as well."""
     h: torch.Tensor
     norm: Optional[Norm]
     res: torch.Tensor
+    shifted: bool = False
+
+
+@dataclass
+class BranchPair:
+    """What a mixer that says `emits_pair` returns: two branches still to be joined,
+    factor * (first / rms(first) * w_first + second / rms(second) * w_second), by the kernel that ends the branch."""
+    first: torch.Tensor
+    second: torch.Tensor
+    w_first: torch.Tensor      # float32 [width]
+    w_second: torch.Tensor
+    eps: float
+    factor: float
 
 
 class StreamEntry(Part):
@@ -270,6 +285,10 @@ class PositionEncoding(Part):
         cache-write kernel can apply itself; None otherwise."""
         return None
 
+    def rotary_multiplier(self) -> float:
+        """What cos and sin of `fused_rotary` are multiplied by."""
+        return 1.0
+
     def score_slopes(self) -> Optional[torch.Tensor]:
         """float32 [query heads] when the encoding is a bias on the attention scores that grows with distance,
         slope * (key position - query position); None otherwise."""
@@ -282,8 +301,14 @@ class PositionEncoding(Part):
 
 
 class Shift(Part):
-    """Mixes every token's row with the row of the token before it in the same request, which is the request's state between
+    """Mixes every token's row with rows of the tokens before it in the same request, which are the request's state between
     steps: `state_spec()` says what a slot holds, `forward(ctx, h, state) -> h'` reads and updates it."""
+
+    def single_token_filter(self) -> Optional[torch.Tensor]:
+        """float32 [width, taps] when the part is h + sum_j f[:, j] * (rows of the tokens before and the token's own, oldest
+        first) with the rows before, float32 [taps - 1, width], as its state: a step of single tokens may then have it done by the
+        kernel that norms the rows.  None otherwise."""
+        return None
 
     def state_spec(self) -> StateSpec:
         raise NotImplementedError
@@ -299,6 +324,7 @@ class Mixer(Part):
     fuses_norm = False
     # what the block multiplies the output by where it adds it to the stream; only blocks that say `scales_mixer` do
     out_scale = 1.0
+    emits_pair = False          # `forward` returns a `BranchPair`; only blocks that say `takes_pair` join one
 
     def cache_spec(self) -> Optional[KVCacheSpec]:
         return None
@@ -347,8 +373,16 @@ class Block:
         and may return a `Prenormed` for that norm as x.  None (the default): the block wants a plain tensor."""
         return None
 
+    def entry_shift(self) -> Optional["Shift"]:
+        """The `Shift` that the block's first norm's output passes (its state is `LayerCache.extra[self.entry_shift_role]`), for a
+        block before it that says `fuses_next_shift`: its `forward` is then also called with `next_shift=` (part, state)."""
+        return None
+
+    entry_shift_role = "mixer_shift"
     fuses_next_norm = False
+    fuses_next_shift = False
     scales_mixer = False        # the block multiplies its mixer's output by `Mixer.out_scale`
+    takes_pair = False          # the block joins a mixer's `BranchPair`
 
 
 # ----------------------------------------------------------------------------- registries

@@ -12,12 +12,17 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from .. import kernels
-from .base import Block, LayerCache, Norm, NormAfter, Normed, Part, StepContext, register_part
+from .base import Block, BranchPair, LayerCache, Norm, NormAfter, Normed, Part, Shift, StepContext, register_part
 
 # A step of a few tokens in bfloat16: a norm between two weight-streaming products is done by those products
 # (the one before adds to the residual stream and leaves sums of squares, the one after divides).  LMSF_FUSE_NORMS=0:
 # every norm is a kernel of its own.
 FUSE_NORMS = os.environ.get("LMSF_FUSE_NORMS", "1") != "0"
+
+
+def divides_rows(norm: Optional[Norm]) -> bool:
+    """Whether a norm is a division by the root mean square and one weight: what the kernels that end a block apply."""
+    return hasattr(norm, "weight_f32") and not norm.centred and not getattr(norm, "has_layer_scale", False)
 
 
 def norm_after(ctx: StepContext, producer: Part, norm: Norm, consumer: Part, res: Optional[torch.Tensor]) -> Optional[NormAfter]:
@@ -60,56 +65,84 @@ class SandwichNormBlock(Block):
     may carry a layer scale (a learned vector that multiplies its output).  The residual stream is float32 and every
     sum into it is made in float32 from the float32 normed branch (the branch is never rounded before it is added).
     One kernel does what lies between two branches: the post norm of the branch before, the add, and the pre norm of
-    the branch after (`kernels.stream_norm`); with `next_entry` it also applies the next block's first norm and
-    hands it over as a `Normed`.  A layer may have no feed-forward.  With a `mixer_shift` the mixer reads the first norm's
-    output mixed with the row of the token before (a `Shift` part, whose state per request the block declares)."""
+    the branch after (`kernels.stream_norm`, or `kernels.stream_layer` where a norm takes the mean off); with `next_entry` it
+    also applies the next block's first norm and hands it over as a `Normed`.  A layer may have no feed-forward.  With a
+    `mixer_shift` or a `ffn_shift` the mixer or the feed-forward reads its norm's output mixed with rows of the tokens before (a
+    `Shift` part, whose state per request the block declares); in a step of single tokens a shift that is a short filter is part
+    of the kernel that norms the rows.  A mixer may return a `BranchPair`, which the same kernel joins."""
     ROLES = {"mixer_norm": "norm", "mixer_shift": "shift", "mixer": "mixer", "mixer_post_norm": "norm",
-             "ffn_norm": "norm", "feed_forward": "feed_forward", "ffn_post_norm": "norm"}
-    OPTIONAL_ROLES = ("mixer_shift", "ffn_norm", "feed_forward", "ffn_post_norm")
+             "ffn_norm": "norm", "ffn_shift": "shift", "feed_forward": "feed_forward", "ffn_post_norm": "norm"}
+    OPTIONAL_ROLES = ("mixer_shift", "ffn_norm", "ffn_shift", "feed_forward", "ffn_post_norm")
     fuses_next_norm = True
+    fuses_next_shift = True
+    takes_pair = True
 
     def __init__(self, parts: Dict[str, Part]):
         super().__init__(parts)
         self.mixer_norm, self._mixer, self.mixer_post = parts["mixer_norm"], parts["mixer"], parts["mixer_post_norm"]
-        self.mixer_shift = parts.get("mixer_shift")
+        self.mixer_shift, self.ffn_shift = parts.get("mixer_shift"), parts.get("ffn_shift")
         self.feed_forward = parts.get("feed_forward")
         self.ffn_norm, self.ffn_post = parts.get("ffn_norm"), parts.get("ffn_post_norm")
         if self.feed_forward is not None and (self.ffn_norm is None or self.ffn_post is None):
             raise ValueError("a feed-forward needs the norms before and after it")
         for n in (self.mixer_norm, self.mixer_post, self.ffn_norm, self.ffn_post):
             if n is not None and not hasattr(n, "weight_f32"):
-                raise ValueError("the sandwich block takes norms that are a factor per row times a weight (rmsnorm)")
+                raise ValueError("the sandwich block takes norms that are a factor per row times a weight (rmsnorm, layernorm)")
 
     def entry(self) -> Optional[Tuple[Norm, Part]]:
         return self.mixer_norm, self._mixer
 
+    def entry_shift(self) -> Optional[Shift]:
+        return self.mixer_shift
+
     def state_specs(self):
-        return {"mixer_shift": self.mixer_shift.state_spec()} if self.mixer_shift is not None else {}
+        return {role: p.state_spec() for role, p in (("mixer_shift", self.mixer_shift), ("ffn_shift", self.ffn_shift)) if p is not None}
 
     @staticmethod
-    def _between(res: torch.Tensor, branch: torch.Tensor, post, nxt: Optional[Norm]):
-        """res += post(branch); returns nxt(res) in the branch's type (None without nxt)."""
-        h = torch.empty_like(branch) if nxt is not None else None
+    def _between(ctx: StepContext, res: torch.Tensor, branch, post: Optional[Norm], nxt: Optional[Norm], shift=None):
+        """res += post(branch) (if there is a branch: a tensor or a pair); returns (nxt(res) in the activation type, None without
+        nxt; whether it has passed `shift`, a (part, state) behind nxt, as well)."""
+        filt = None
+        if shift is not None and nxt is not None and FUSE_NORMS and ctx.decode_only and ctx.n_tokens == ctx.n_seqs:
+            f = shift[0].single_token_filter()
+            filt = (f, shift[1], ctx.state_slot) if f is not None else None
+        pair = branch if isinstance(branch, BranchPair) else None
+        y = branch.first if pair is not None else branch
+        h = torch.empty(res.shape, dtype=ctx.dtype, device=res.device) if nxt is not None else None
+        if pair is not None or filt is not None or branch is None or post.centred or (nxt is not None and nxt.centred):
+            if post is not None and getattr(post, "has_layer_scale", False):
+                raise ValueError("a layer scale is not built with norms that take the mean off, pairs of branches and filters")
+            kernels.stream_layer(res, y=y, pair=(pair.second, pair.w_first, pair.w_second, pair.eps, pair.factor) if pair is not None else None,
+                                 w_post=post.weight_f32() if y is not None else None, eps_post=post.eps if y is not None else 0.0,
+                                 post_centred=y is not None and post.centred, h=h, w_next=nxt.weight_f32() if nxt is not None else None,
+                                 eps_next=nxt.eps if nxt is not None else 0.0, next_centred=nxt is not None and nxt.centred, filt=filt)
+            return h, filt is not None
         kernels.stream_norm(res, y=branch, w_post=post.weight_f32(), layer_scale=post.scale_f32(), eps_post=post.eps,
                             h=h, w_next=nxt.weight_f32() if nxt is not None else None,
                             eps_next=nxt.eps if nxt is not None else 0.0)
-        return h
+        return h, False
 
     def forward(self, ctx: StepContext, x, res: Optional[torch.Tensor], cache: LayerCache,
-                next_entry: Optional[Tuple[Norm, Part]] = None):
-        h, res = self.mixer_norm.forward_residual(x, res)      # x: None (complete stream), a Normed, or a pending branch
-        if self.mixer_shift is not None:
-            h = self.mixer_shift.forward(ctx, h, cache.extra["mixer_shift"])
+                next_entry: Optional[Tuple[Norm, Part]] = None, next_shift=None):
+        own = [(p, cache.extra[role]) if p is not None else None for role, p in (("mixer_shift", self.mixer_shift), ("ffn_shift", self.ffn_shift))]
+        if x is None and own[0] is not None and own[0][0].single_token_filter() is not None:      # a complete stream
+            h, shifted = self._between(ctx, res, None, None, self.mixer_norm, own[0])
+        else:
+            shifted = isinstance(x, Normed) and x.shifted
+            h, res = self.mixer_norm.forward_residual(x, res)      # x: None (complete stream), a Normed, or a pending branch
+        if own[0] is not None and not shifted:
+            h = own[0][0].forward(ctx, h, own[0][1])
         a = self._mixer.forward(ctx, h, cache)
         nxt = next_entry[0] if next_entry is not None and hasattr(next_entry[0], "weight_f32") and \
             not getattr(next_entry[0], "has_layer_scale", False) else None
-        if self.feed_forward is None:
-            h = self._between(res, a, self.mixer_post, nxt)
-            return (Normed(h, nxt, res) if nxt is not None else None), res
-        h = self._between(res, a, self.mixer_post, self.ffn_norm)
-        f = self.feed_forward.forward(ctx, h)
-        h = self._between(res, f, self.ffn_post, nxt)
-        return (Normed(h, nxt, res) if nxt is not None else None), res
+        post = self.mixer_post
+        if self.feed_forward is not None:
+            h, shifted = self._between(ctx, res, a, post, self.ffn_norm, own[1])
+            if own[1] is not None and not shifted:
+                h = own[1][0].forward(ctx, h, own[1][1])
+            a, post = self.feed_forward.forward(ctx, h), self.ffn_post
+        h, shifted = self._between(ctx, res, a, post, nxt, next_shift)
+        return (Normed(h, nxt, res, shifted) if nxt is not None else None), res
 
 
 @register_part("block", "branch_norm")
@@ -136,7 +169,7 @@ class BranchNormBlock(Block):
                     raise ValueError(f"the branch {role!r} needs its norm {norm!r}")
                 self.branches.append((parts[role], parts[norm]))
         for _, n in self.branches:
-            if not hasattr(n, "weight_f32") or getattr(n, "has_layer_scale", False):
+            if not divides_rows(n):
                 raise ValueError("the branch-norm block takes norms that are a factor per row times a weight (rmsnorm)")
 
     def entry(self) -> Optional[Tuple[Norm, Part]]:
@@ -196,7 +229,7 @@ class ParallelGatedBlock(Block):
         super().__init__(parts)
         self.norm, self._mixer, self.gates = parts["norm"], parts["mixer"], parts["gates"]
         self.feed_forward = parts.get("feed_forward")
-        if not hasattr(self.norm, "weight_f32") or getattr(self.norm, "has_layer_scale", False):
+        if not divides_rows(self.norm):
             raise ValueError("the parallel block takes a norm that is a factor per row times a weight (rmsnorm)")
         branches = 2 if self.feed_forward is not None else 1
         if not hasattr(self.gates, "logits") or self.gates.out_features != branches * self.norm.hidden_size:
@@ -218,8 +251,7 @@ class ParallelGatedBlock(Block):
         z = self.gates.logits(h)
         a = self._mixer.forward(ctx, h, cache)
         f = self.feed_forward.forward(ctx, h) if self.feed_forward is not None else None
-        nxt = next_entry[0] if next_entry is not None and hasattr(next_entry[0], "weight_f32") and \
-            not getattr(next_entry[0], "has_layer_scale", False) else None
+        nxt = next_entry[0] if next_entry is not None and divides_rows(next_entry[0]) else None
         h_next = torch.empty_like(a) if nxt is not None else None
         kernels.gated_branches(res, z, self.gates.bias_f32(), a, f, h=h_next,
                                w_next=nxt.weight_f32() if nxt is not None else None,
@@ -246,7 +278,7 @@ class ParallelNormsBlock(Block):
         if (self.feed_forward is None) != (self.ffn_norm is None):
             raise ValueError("a feed-forward and its norm go together")
         for n in (self.mixer_norm, self.ffn_norm):
-            if n is not None and (not hasattr(n, "weight_f32") or getattr(n, "has_layer_scale", False)):
+            if n is not None and not divides_rows(n):
                 raise ValueError("the block takes norms that are a factor per row times a weight (rmsnorm)")
         if self.ffn_norm is not None and self.ffn_norm.eps != self.mixer_norm.eps:
             raise ValueError("the block's two norms share one eps")
@@ -286,7 +318,7 @@ class ParallelNormsBlock(Block):
             n = next_entry[0]
             if isinstance(n, ParallelNorms):
                 norms = n
-            elif hasattr(n, "weight_f32") and not getattr(n, "has_layer_scale", False):
+            elif divides_rows(n):
                 norms = ParallelNorms(n, None)
         h1, h2 = self._end(ctx, res, a, self._mixer.out_scale, f, norms)
         if norms is None:

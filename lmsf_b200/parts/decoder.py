@@ -38,6 +38,8 @@ class DecoderModel:
             m = self.blocks[-1].mixer
             if m is not None and m.out_scale != 1.0 and not cls.scales_mixer:
                 raise ValueError(f"block {ls.block!r} does not multiply its mixer's output, which asks for a factor {m.out_scale}")
+            if m is not None and m.emits_pair and not cls.takes_pair:
+                raise ValueError(f"block {ls.block!r} does not join the pair of branches that its mixer returns")
         self.final_norm = build_part("norm", spec.final_norm)
         self.lm_head = build_part("linear", spec.lm_head)
         self._owned += [*with_nested(self.final_norm, spec.final_norm), *with_nested(self.lm_head, spec.lm_head)]
@@ -106,12 +108,15 @@ class DecoderModel:
                     res = replaced
             # a block that can take the next block's first norm into its last product is told that norm and its reader
             # (not across an entry that changes the stream in between)
-            entry = None
+            entry, more = None, {}
             if block.fuses_next_norm and j + 1 < len(self.calls) and self.calls[j + 1].entry is None:
-                entry = self.blocks[self.calls[j + 1].layer].entry()
+                nxt = self.blocks[self.calls[j + 1].layer]
+                entry = nxt.entry()
+                if block.fuses_next_shift and nxt.entry_shift() is not None:
+                    more = {"next_shift": (nxt.entry_shift(), caches[j + 1].extra[nxt.entry_shift_role])}
             with span(f"layer {call.layer}"):
                 if entry is not None:
-                    x, res = block.forward(ctx, x, res, caches[j], next_entry=entry)
+                    x, res = block.forward(ctx, x, res, caches[j], next_entry=entry, **more)
                 else:
                     x, res = block.forward(ctx, x, res, caches[j])
             if self.layer_hook is not None:

@@ -1,4 +1,4 @@
-"""RMSNorm, alone or fused with the residual add before it.
+"""RMSNorm, alone or fused with the residual add before it, and a layer norm of the float32 stream.
 
 Formula of the reference: vllm/kernels/layernorm_kernels.cu:13-68, called from
 core/src/model_executor/models/llama/llama.rs:295-317, :333, :461-462.  The residual stream is
@@ -107,3 +107,54 @@ class RMSNorm(Norm):
         h = torch.empty_like(p.x)
         kernels.finish_rmsnorm(h, p.res, p.sumsq, self.weight, self.eps)
         return h
+
+
+@register_part("norm", "layernorm")
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * w, no bias; float32 inside (csrc/layer_norm.cu)."""
+    graph_safe = True
+    centred = True
+    has_layer_scale = False
+
+    def __init__(self, hidden_size: int, eps: float):
+        self.hidden_size, self.eps = int(hidden_size), float(eps)
+        self.weight: Optional[torch.Tensor] = None
+        self._w32: Optional[torch.Tensor] = None
+        self._act_dtype: Optional[torch.dtype] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {"weight": WeightSpec([(self.hidden_size,)], keep_fp32=True)}
+
+    def prepare(self, dtype, device) -> None:
+        self._act_dtype, self._w32 = dtype, None
+        self.weight_f32()
+
+    def weight_f32(self) -> torch.Tensor:
+        if self._w32 is None or self._w32.device != self.weight.device:
+            self._w32 = self.weight.float().contiguous()
+        return self._w32
+
+    def of_stream(self, res: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+        """The norm of a complete float32 stream, in the activation type."""
+        h = torch.empty(res.shape, dtype=dtype, device=res.device)
+        kernels.stream_layer(res, h=h, w_next=self.weight_f32(), eps_next=self.eps, next_centred=True)
+        return h
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        res = x
+        if x.dtype != torch.float32:
+            res = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+            kernels.stream_begin(res, x)
+        return self.of_stream(res.contiguous(), x.dtype)
+
+    def forward_residual(self, x: Union[torch.Tensor, Normed, None], res: Optional[torch.Tensor]) -> Tuple[torch.Tensor, torch.Tensor]:
+        if isinstance(x, Normed):
+            if x.norm is not self or x.res is not res:
+                raise ValueError("a Normed activation was prepared for another norm or residual stream")
+            return x.h, res
+        if x is not None and res is None:        # x starts the stream
+            res = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+            kernels.stream_begin(res, x)
+        elif x is not None:
+            kernels.stream_branches(res, x)
+        return self.of_stream(res, x.dtype if x is not None else (self._act_dtype or torch.float32)), res

@@ -1,4 +1,6 @@
-"""Two mixers side by side that read the same input and whose outputs are added with a factor each:
+"""Two mixers side by side that read the same input.
+
+`parallel_mixers`: their outputs are added with a factor each,
 
   out = left_scale * attention(h) + right_scale * memory(h)
 
@@ -7,14 +9,22 @@ are on the device: one product for everything that reads h (queries, keys, and t
 output projections ([left | right] side by side).  The right factor is applied to the memory's float32 output before it is
 rounded; the left one is asked of the block (`Mixer.out_scale`), which adds the result to the float32 stream: nothing is
 rounded on its account.  The pages of the cache are the left mixer's, the state slot the right one's.
+
+`normed_parallel_mixers`: each output is divided by its root mean square over the width and multiplied by a weight of its own,
+
+  out = factor * (left / rms(left) * w_left + right / rms(right) * w_right)
+
+The left one is attention whose queries and keys pass a filter, the right one a selective state space.  What reads h is one product
+again; the two output products stay apart, and the block's kernel joins them (`BranchPair`): nothing is rounded between the two
+norms and the sum into the stream.  A state slot holds the right mixer's state and behind it the left one's carried inputs.
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import Dict, Optional
 
 import torch
 
-from .base import KVCacheSpec, LayerCache, Mixer, StateSpec, StepContext, register_part
+from .base import BranchPair, KVCacheSpec, LayerCache, Mixer, StateSpec, StepContext, WeightSpec, register_part
 from .linear import matmul_tn
 
 
@@ -77,3 +87,61 @@ class ParallelMixers(Mixer):
         n = L.q_size + L.kv_size
         R.mix_projected(ctx, p[:, n:n + R.in_size], cache, y[:, a:a + b], self.right_factor)
         return matmul_tn(y, self._out)
+
+
+@register_part("mixer", "normed_parallel_mixers")
+class NormedParallelMixers(Mixer):
+    graph_safe = True
+    emits_pair = True
+
+    def __init__(self, mixer_left: Mixer, mixer_right: Mixer, eps: float, factor: float = 0.5):
+        left, right = mixer_left, mixer_right
+        if not getattr(left, "qk_filter_taps", 0) or not hasattr(right, "state_floats") or not hasattr(right, "mix_projected") \
+                or left.hidden_size != right.hidden_size:
+            raise ValueError("side by side stand attention with filtered queries and keys (left) and a selective state space (right) of one width")
+        if left.has_out_bias:
+            raise ValueError("mixers side by side are not built with a bias of the output projection")
+        self.left, self.right = left, right
+        self.hidden_size, self.eps, self.factor = left.hidden_size, float(eps), float(factor)
+        self.left_at = (right.state_floats() + 3) // 4 * 4          # where a slot's left part starts (16-byte aligned)
+        self.left_norm: Optional[torch.Tensor] = None
+        self.right_norm: Optional[torch.Tensor] = None
+        self._w_left: Optional[torch.Tensor] = None
+        self._w_right: Optional[torch.Tensor] = None
+        self._in: Optional[torch.Tensor] = None
+        self._in_bias: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {n: WeightSpec([(self.hidden_size,)], keep_fp32=True) for n in ("left_norm", "right_norm")}
+
+    def cache_spec(self) -> Optional[KVCacheSpec]:
+        return self.left.cache_spec()
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec(((self.left_at + self.left.filter_state_floats() + 3) // 4 * 4,))
+
+    def activation_width(self) -> int:
+        return self.left.activation_width() + self.right.activation_width() + 2 * self.hidden_size
+
+    def prepare(self, dtype, device) -> None:
+        self._w_left, self._w_right = self.left_norm.float().contiguous(), self.right_norm.float().contiguous()
+        L, R = self.left, self.right
+        if self._in is not None and self._in.device == L.qkv.device and L.qkv.data_ptr() == self._in.data_ptr():
+            return
+        n, rows = L.qkv.shape[0], L.qkv.shape[0] + R.in_proj.shape[0]
+        pad = -rows % 16                                   # rows of the product stay 16-byte aligned
+        self._in = torch.cat([L.qkv, R.in_proj, L.qkv.new_zeros((pad, L.qkv.shape[1]))], 0).contiguous()
+        self._in_bias = None
+        if L.qkv_bias is not None:
+            self._in_bias = torch.cat([L.qkv_bias, L.qkv_bias.new_zeros(rows + pad - n)], 0).contiguous()
+        L.qkv, R.in_proj = self._in[:n], self._in[n:rows]  # the parts' own matrices become views of the merged one
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> BranchPair:
+        L, R = self.left, self.right
+        n = L.q_size + L.kv_size
+        p = matmul_tn(h, self._in, bias=self._in_bias)
+        a = torch.empty((ctx.n_tokens, L.q_size), dtype=p.dtype, device=p.device)
+        b = torch.empty((ctx.n_tokens, R.inner), dtype=p.dtype, device=p.device)
+        L.attend_filtered(ctx, p[:, :n], cache, a, self.left_at)
+        R.mix_projected(ctx, p[:, n:n + R.in_size], cache, b)
+        return BranchPair(matmul_tn(a, L.o), matmul_tn(b, R.o), self._w_left, self._w_right, self.eps, self.factor)

@@ -68,8 +68,11 @@ class SelectiveStateSpace(_StateMatrixMixer):
                 "skip": WeightSpec([(H,)], keep_fp32=True), "norm": WeightSpec([(self.inner,)], keep_fp32=True),
                 "o": WeightSpec([(self.hidden_size, self.inner)])}
 
+    def state_floats(self) -> int:
+        return self.matrix_floats + (self.taps - 1) * self.channels
+
     def state_spec(self) -> Optional[StateSpec]:
-        return StateSpec((self.matrix_floats + (self.taps - 1) * self.channels,))
+        return StateSpec((self.state_floats(),))
 
     def activation_width(self) -> int:
         return self.in_size + self.channels + 3 * self.inner
@@ -77,9 +80,10 @@ class SelectiveStateSpace(_StateMatrixMixer):
     def prepare(self, dtype, device) -> None:
         self._f32 = {n: getattr(self, n).float().contiguous() for n in ("conv", "conv_bias", "dt_bias", "a_log", "skip", "norm")}
 
-    def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
+    def mix_projected(self, ctx: StepContext, p: torch.Tensor, cache: LayerCache, out: torch.Tensor) -> None:
+        """From the rows of the input product (a view [n, in_size]) to what the output projection reads, in `out` (a view [n,
+        inner])."""
         n, I, GN, H = ctx.n_tokens, self.inner, self.groups * self.state_size, self.num_heads
-        p = matmul_tn(h, self.in_proj)
         z, xbc, dt = p[:, :I], p[:, I:I + self.channels], p[:, I + self.channels:]
         c = torch.empty((n, self.channels), dtype=p.dtype, device=p.device)
         w = self._f32
@@ -89,8 +93,12 @@ class SelectiveStateSpace(_StateMatrixMixer):
         kernels.gated_scan(y, c[:, I + GN:], c[:, I:I + GN], c[:, :I], dt, None, w["dt_bias"], w["a_log"], w["skip"],
                            cache.state, ctx.cu_q, ctx.state_slot, ctx.n_seqs, H, self.groups, self.state_size, self.head_dim,
                            delta=False, k_times_dt=True)
-        g = torch.empty((n, I), dtype=p.dtype, device=p.device)
-        kernels.grouped_gated_norm(g, y, z, w["norm"], I // self.norm_groups, self.eps, gate_act="silu", gate_first=True)
+        kernels.grouped_gated_norm(out, y, z, w["norm"], I // self.norm_groups, self.eps, gate_act="silu", gate_first=True)
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
+        p = matmul_tn(h, self.in_proj)
+        g = torch.empty((ctx.n_tokens, self.inner), dtype=p.dtype, device=p.device)
+        self.mix_projected(ctx, p, cache, g)
         return matmul_tn(g, self.o)
 
 

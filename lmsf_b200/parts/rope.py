@@ -20,7 +20,7 @@ from .base import ANY_SIZE, PositionEncoding, StepContext, WeightSpec, register_
 
 def rope_inverse_frequencies(rot_dim: int, theta: float, scaling_type: str = "default", factor: float = 1.0,
                              low_freq_factor: float = 1.0, high_freq_factor: float = 4.0,
-                             original_max_position_embeddings: int = 8192, beta_fast: float = 32.0,
+                             original_max_position_embeddings: float = 8192, beta_fast: float = 32.0,
                              beta_slow: float = 1.0) -> List[float]:
     """f_i = theta^(-2i/rot_dim), then by scaling type:
     linear: f_i / factor.
@@ -66,14 +66,16 @@ class RotaryEmbedding(PositionEncoding):
 
     def __init__(self, rot_dim: int, theta: float = 10000.0, is_neox: bool = True, scaling_type: str = "default",
                  factor: float = 1.0, low_freq_factor: float = 1.0, high_freq_factor: float = 4.0,
-                 original_max_position_embeddings: int = 8192):
+                 original_max_position_embeddings: float = 8192, beta_fast: float = 32.0, beta_slow: float = 1.0):
         if rot_dim <= 0 or rot_dim % 2:
             raise ValueError(f"rotary width must be a positive even number, got {rot_dim}")
         self.rot_dim = int(rot_dim)
         self.is_neox = bool(is_neox)
         self.inv_freq_host = rope_inverse_frequencies(rot_dim, float(theta), scaling_type, float(factor),
                                                       float(low_freq_factor), float(high_freq_factor),
-                                                      int(original_max_position_embeddings))
+                                                      original_max_position_embeddings, float(beta_fast), float(beta_slow))
+        # what cos and sin are multiplied by (only parts that say so take a rotation that also stretches)
+        self.mult = yarn_magnitude(float(factor)) if scaling_type == "yarn" else 1.0
         self.inv_freq: Optional[torch.Tensor] = None
 
     def prepare(self, dtype: torch.dtype, device: torch.device) -> None:
@@ -81,6 +83,9 @@ class RotaryEmbedding(PositionEncoding):
 
     def fused_rotary(self) -> Optional[Tuple[torch.Tensor, int, bool]]:
         return self.inv_freq, self.rot_dim, self.is_neox
+
+    def rotary_multiplier(self) -> float:
+        return self.mult
 
     def apply(self, ctx: StepContext, q, k, n_q_heads, n_kv_heads, head_dim) -> None:
         kernels.rope_cache_write(q, None, None, ctx.positions, None, None, 0, None, self.inv_freq, self.rot_dim,
