@@ -211,6 +211,7 @@ struct ScanArgs {
   float unit_eps, q_scale;
   float* qf; float* kf; float4* gates;                         // what scan_prepare leaves for the scan (below)
   int n_tokens;
+  const int* seq_ids;                                          // requests that are scanned (null: all)
 };
 
 constexpr int kScanCols = 32;       // columns of the state per block
@@ -275,7 +276,7 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(ScanArgs a) {
   __shared__ float sv[CH][COLS];
   __shared__ float4 sg[CH];
   const int tid = threadIdx.x, c = tid / R, r = tid % R;
-  const int head = blockIdx.y, seq = blockIdx.z, col = blockIdx.x * COLS + c;
+  const int head = blockIdx.y, seq = a.seq_ids ? a.seq_ids[blockIdx.z] : blockIdx.z, col = blockIdx.x * COLS + c;
   const int g = head / (a.H / a.G);
   const int t0 = a.cu_q[seq], n = a.cu_q[seq + 1] - t0;
   if (n <= 0) return;
@@ -500,12 +501,13 @@ LMSF_API long long lmsf_gated_scan_scratch_floats(int n_tokens, int H, int G, in
   return (long long)n_tokens * (2LL * G * lmsf::scan_row_floats(dk) + 4LL * H);
 }
 
+// seq_ids (may be null): n_seqs requests among those of cu_q that are scanned; the others are left alone.
 LMSF_API int lmsf_gated_scan(float* out, long long out_stride, const void* q, const void* k, const void* v, long long q_stride,
                              long long k_stride, long long v_stride, const void* dt, long long dt_stride, const void* beta,
                              long long beta_stride, const float* dt_bias, const float* a_log, const float* skip, float* state,
                              long long slot_stride, const int* cu_q, const int* state_slot, int n_seqs, int n_tokens, int H,
                              int G, int dk, int dv, int delta, int k_times_dt, int unit_qk, float unit_eps, float q_scale,
-                             float* scratch, int dtype, void* stream) {
+                             float* scratch, const int* seq_ids, int dtype, void* stream) {
   using namespace lmsf;
   if (n_seqs <= 0 || n_tokens <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > 256 || dv <= 0 || H > 65535 || n_seqs > 65535)
@@ -515,7 +517,7 @@ LMSF_API int lmsf_gated_scan(float* out, long long out_stride, const void* q, co
   const long long rowf = (long long)n_tokens * G * scan_row_floats(dk);
   ScanArgs a{out, out_stride, q, k, v, q_stride, k_stride, v_stride, dt, dt_stride, beta, beta_stride, dt_bias, a_log, skip,
              state, slot_stride, cu_q, state_slot, H, G, dk, dv, k_times_dt, unit_qk, unit_eps, q_scale,
-             scratch, scratch + rowf, reinterpret_cast<float4*>(scratch + 2 * rowf), n_tokens};
+             scratch, scratch + rowf, reinterpret_cast<float4*>(scratch + 2 * rowf), n_tokens, seq_ids};
   cudaStream_t s = (cudaStream_t)stream;
   int rc;
   if (dtype == LMSF_F32) rc = delta ? launch_scan<float, true>(a, n_seqs, s) : launch_scan<float, false>(a, n_seqs, s);

@@ -1055,7 +1055,7 @@ def stream_layer(res: torch.Tensor, y: Optional[torch.Tensor] = None, pair=None,
     _check(rc, "layer_norm.cu", "lmsf_layer_norm")
 
 
-def conv_rope_cache_write(q: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, state_offset: int,
+def conv_rope_cache_write(q: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], state_offset: int,
                           cu_q: torch.Tensor, state_slot: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor,
                           block_size: int, cache: torch.Tensor, inv_freq: Optional[torch.Tensor], rot_dim: int, mult: float,
                           n_q_heads: int, n_kv_heads: int, head_dim: int, n_seqs: int, max_q: int,
@@ -1072,8 +1072,8 @@ def conv_rope_cache_write(q: torch.Tensor, x: torch.Tensor, w: torch.Tensor, sta
     _rows(q, n_q_heads * head_dim, "conv_rope: q", x.dtype)
     if w.dtype != torch.float32 or w.shape != (taps, C) or not w.is_contiguous():
         raise KernelError("conv_rope: w must be contiguous float32 [taps, channels]")
-    if state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state_offset < 0 or \
-            state_offset + (taps - 1) * C > state.shape[1]:
+    if taps > 1 and (state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state_offset < 0 or
+                     state_offset + (taps - 1) * C > state.shape[1]):
         raise KernelError("conv_rope: the state must be contiguous float32 [slots, size] with room for [taps - 1, channels]")
     if cache.dtype != x.dtype or not cache.is_contiguous() or tuple(cache.shape[1:]) != (2, n_kv_heads, block_size, head_dim):
         raise KernelError(f"conv_rope: cache of shape {tuple(cache.shape)} does not match [pages, 2, {n_kv_heads}, {block_size}, {head_dim}] of {x.dtype}")
@@ -1083,7 +1083,8 @@ def conv_rope_cache_write(q: torch.Tensor, x: torch.Tensor, w: torch.Tensor, sta
               [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
                c_void_p, c_void_p])
-    rc = f(_ptr(x), x.stride(0), _ptr(q), q.stride(0), _ptr(w), taps, _ptr(state) + 4 * state_offset, state.stride(0),
+    rc = f(_ptr(x), x.stride(0), _ptr(q), q.stride(0), _ptr(w), taps, _ptr(state) + 4 * state_offset if taps > 1 else None,
+           state.stride(0) if taps > 1 else 0,
            _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), _i32(positions, "positions"), _i32(block_table, "block_table"),
            block_table.shape[1], block_size, _ptr(cache), cache.stride(0), _ptr(inv_freq), rot_dim, float(mult), n_q_heads, n_kv_heads,
            head_dim, n_seqs, int(max_q), dtype_code(x.dtype), _i32(error_flag, "error_flag"), _stream())
@@ -1237,14 +1238,17 @@ def gated_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
                beta: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, skip: Optional[torch.Tensor],
                state: torch.Tensor, cu_q: torch.Tensor, state_slot: torch.Tensor, n_seqs: int, heads: int, qk_heads: int,
                dk: int, dv: int, delta: bool, k_times_dt: bool = False, unit_qk: bool = False, unit_eps: float = 1e-6,
-               q_scale: float = 1.0):
+               q_scale: float = 1.0, seq_ids: Optional[torch.Tensor] = None):
     """Per request, head h and token: step = softplus(dt[t, h] + dt_bias[h]), a = exp(-exp(a_log[h]) * step);
     plain rule: S = a S + (step k) v^T (k v^T without k_times_dt); delta rule: S = a S, u = sigmoid(beta[t, h]) (v - S^T k),
     S += k u^T; out[t, h] = S^T q + skip[h] v.  Head h reads q/k head h // (heads / qk_heads); unit_qk makes q and k unit
     vectors first (x / sqrt(sum x^2 + unit_eps)) and multiplies q by q_scale.  S = the first heads * dv * dk values of
     state[slot] (float32 [slots, size], stored [head][dv][dk]), read before and written after.
     q, k: [n, qk_heads * dk]; v: [n, heads * dv]; dt, beta: [n, heads] (views of one dtype); out: float32 [n, heads * dv].
-    Two launches: one prepares q, k and the tokens' decays in a scratch that this function allocates, one scans."""
+    Two launches: one prepares q, k and the tokens' decays in a scratch that this function allocates, one scans.
+    seq_ids (int32): the requests that are scanned, all without it."""
+    if seq_ids is not None:
+        n_seqs = seq_ids.numel()
     n = q.shape[0]
     _rows(q, qk_heads * dk, "gated_scan: q")
     _rows(k, qk_heads * dk, "gated_scan: k", q.dtype)
@@ -1258,7 +1262,7 @@ def gated_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
     f = _func("recurrent.cu", "lmsf_gated_scan",
               [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong,
                c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int,
-               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p])
+               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_void_p])
     need = _func("recurrent.cu", "lmsf_gated_scan_scratch_floats", [c_int, c_int, c_int, c_int])
     need.restype = c_longlong
     scratch = torch.empty(int(need(n, heads, qk_heads, dk)), dtype=torch.float32, device=q.device)
@@ -1266,9 +1270,50 @@ def gated_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
            _ptr(beta), beta.stride(0) if beta is not None else 0, _f32vec(dt_bias, heads, "dt_bias"),
            _f32vec(a_log, heads, "a_log"), _f32vec(skip, heads, "skip"), _ptr(state), state.stride(0), _i32(cu_q, "cu_q"),
            _i32(state_slot, "state_slot"), n_seqs, n, heads, qk_heads, dk, dv, int(delta), int(k_times_dt), int(unit_qk),
-           float(unit_eps), float(q_scale), _ptr(scratch), dtype_code(q.dtype), _stream())
+           float(unit_eps), float(q_scale), _ptr(scratch), _i32(seq_ids, "seq_ids"), dtype_code(q.dtype), _stream())
     _check(rc, "recurrent.cu", "lmsf_recurrent")
     add_launches(1)                                            # two launches: prepare and scan
+
+
+def scan_chunk_tokens() -> int:
+    """Tokens of a chunk of `scan_chunks`."""
+    return _func("scan_chunks.cu", "lmsf_scan_chunk_tokens", [])()
+
+
+def scan_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor,
+                a_log: torch.Tensor, skip: Optional[torch.Tensor], state: torch.Tensor, cu_q: torch.Tensor, state_slot: torch.Tensor,
+                n_seqs: int, heads: int, qk_heads: int, dk: int, dv: int, items: Optional[torch.Tensor] = None,
+                spans: Optional[torch.Tensor] = None):
+    """The plain rule of `gated_scan` with k_times_dt on the same state.  items, spans None: every request brings one token, one
+    launch.  Else items (int32 [chunks, 4]: request, first token, end token, chunk number) cut long portions into chunks of at most
+    `scan_chunk_tokens()` tokens and spans (int32 [portions, 4]: request, first item, end item, 0) name each portion's chunks; four
+    launches over a scratch that this function allocates."""
+    _rows(q, qk_heads * dk, "scan_chunks: q")
+    _rows(k, qk_heads * dk, "scan_chunks: k", q.dtype)
+    _rows(v, heads * dv, "scan_chunks: v", q.dtype)
+    _rows(dt, heads, "scan_chunks: dt", q.dtype)
+    _rows(out, heads * dv, "scan_chunks: out", torch.float32)
+    if state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state.shape[1] < heads * dv * dk:
+        raise KernelError("scan_chunks: the state must be contiguous float32 [slots, >= heads * dv * dk]")
+    n_chunks, n_spans, scratch = 0, 0, None
+    if items is not None:
+        if items.dim() != 2 or items.shape[1] != 4 or spans is None or spans.dim() != 2 or spans.shape[1] != 4:
+            raise KernelError("scan_chunks: items and spans are int32 [*, 4]")
+        n_chunks, n_spans = items.shape[0], spans.shape[0]
+        need = _func("scan_chunks.cu", "lmsf_scan_chunks_scratch_floats", [c_int, c_int, c_int, c_int, c_int])
+        need.restype = c_longlong
+        scratch = torch.empty(int(need(n_chunks, heads, qk_heads, dk, dv)), dtype=torch.float32, device=q.device)
+    f = _func("scan_chunks.cu", "lmsf_scan_chunks",
+              [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p,
+               c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+               c_void_p, c_int, c_void_p, c_int, c_void_p])
+    rc = f(_ptr(out), out.stride(0), _ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), _ptr(dt), dt.stride(0),
+           _f32vec(dt_bias, heads, "dt_bias"), _f32vec(a_log, heads, "a_log"), _f32vec(skip, heads, "skip"), _ptr(state), state.stride(0),
+           _i32(cu_q, "cu_q"), _i32(state_slot, "state_slot"), n_seqs, heads, qk_heads, dk, dv, _i32(items, "items"), n_chunks,
+           _i32(spans, "spans"), n_spans, _ptr(scratch), dtype_code(q.dtype), _stream())
+    _check(rc, "scan_chunks.cu", "lmsf_scan_chunks")
+    if n_chunks:
+        add_launches(3)
 
 
 def grouped_gated_norm(out: torch.Tensor, x: torch.Tensor, gate: Optional[torch.Tensor], w: torch.Tensor, group_size: int,

@@ -12,8 +12,9 @@ with the last inputs of a short causal convolution (csrc/recurrent.cu).
   S <- a S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
   out = (norm_head(o) * w * silu(h Wg^T)) Wo^T               (the norm per head, its weight shared by the heads)
 
-Both run prompt portions and single tokens on the same kernels; every index comes from device tensors, so decode steps can
-be replayed from CUDA graphs.  Decays, step sizes, unit norms, the state and every sum of the recurrence are float32; the
+The delta rule runs prompt portions and single tokens on the same kernels; the state space has a launch of its own for single
+tokens and cuts long portions into chunks that run in parallel (csrc/scan_chunks.cu).  Every index of a decode step comes from
+device tensors, so it can be replayed from CUDA graphs.  Decays, step sizes, unit norms, the state and every sum of the recurrence are float32; the
 projections, the convolution and their activation have the activation type.
 """
 from __future__ import annotations
@@ -25,6 +26,34 @@ import torch
 from .. import kernels
 from .base import LayerCache, Mixer, StateSpec, StepContext, WeightSpec, register_part
 from .linear import matmul_tn
+
+LONG_PORTION = 64      # tokens from which a request's portion of the state space is cut into chunks that run in parallel
+CHUNKED = True         # False: everything token by token
+
+
+def portions_plan(ctx: StepContext):
+    """None when no request brings a long portion.  Else (short, chunks, spans), made once a step from the host's copy of the
+    portions' lengths and shared by all layers: `short` lists the requests that are scanned token by token (None if there are
+    none), `chunks` cuts every long portion, `spans` names each portion's chunks."""
+    if not ctx.q_lens or max(ctx.q_lens) < LONG_PORTION:
+        return None
+    plan = ctx.extras.get("state_space_plan")
+    if plan is None:
+        size = kernels.scan_chunk_tokens()
+        short, chunks, spans, t0 = [], [], [], 0
+        for s, n in enumerate(ctx.q_lens):
+            if n >= LONG_PORTION:
+                first = len(chunks)
+                chunks += [(s, c, min(c + size, t0 + n), first + i) for i, c in enumerate(range(t0, t0 + n, size))]
+                spans.append((s, first, len(chunks), 0))
+            else:
+                short.append(s)
+            t0 += n
+        pad = -len(short) % 4
+        flat = torch.tensor(short + [0] * pad + [v for r in chunks + spans for v in r], dtype=torch.int32).to(ctx.device, non_blocking=True)
+        table = flat[len(short) + pad:].view(-1, 4)
+        plan = ctx.extras["state_space_plan"] = (flat[:len(short)] if short else None, table[:len(chunks)], table[len(chunks):])
+    return plan
 
 
 class _StateMatrixMixer(Mixer):
@@ -75,10 +104,28 @@ class SelectiveStateSpace(_StateMatrixMixer):
         return StateSpec((self.state_floats(),))
 
     def activation_width(self) -> int:
-        return self.in_size + self.channels + 3 * self.inner
+        # (a chunk of 64 tokens of a long portion keeps a state per head and a score matrix per group in float32)
+        per_chunk = self.matrix_floats + self.groups * 64 * 64
+        return self.in_size + self.channels + 3 * self.inner + 2 * (per_chunk // 64)
 
     def prepare(self, dtype, device) -> None:
         self._f32 = {n: getattr(self, n).float().contiguous() for n in ("conv", "conv_bias", "dt_bias", "a_log", "skip", "norm")}
+
+    def scan(self, ctx: StepContext, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dt: torch.Tensor, state: torch.Tensor,
+             out: torch.Tensor) -> None:
+        """The recurrence alone, from C, B, x and the raw step sizes to y in float32: single tokens in one launch, portions of
+        LONG_PORTION tokens and more in chunks that run in parallel, what is between token by token."""
+        w = self._f32
+        ends = (w["dt_bias"], w["a_log"], w["skip"], state, ctx.cu_q, ctx.state_slot, ctx.n_seqs, self.num_heads, self.groups, self.state_size,
+                self.head_dim)
+        if CHUNKED and ctx.decode_only:
+            kernels.scan_chunks(out, q, k, v, dt, *ends)
+            return
+        plan = portions_plan(ctx) if CHUNKED else None
+        if plan is None or plan[0] is not None:
+            kernels.gated_scan(out, q, k, v, dt, None, *ends, delta=False, k_times_dt=True, seq_ids=plan[0] if plan is not None else None)
+        if plan is not None:
+            kernels.scan_chunks(out, q, k, v, dt, *ends, items=plan[1], spans=plan[2])
 
     def mix_projected(self, ctx: StepContext, p: torch.Tensor, cache: LayerCache, out: torch.Tensor) -> None:
         """From the rows of the input product (a view [n, in_size]) to what the output projection reads, in `out` (a view [n,
@@ -90,9 +137,7 @@ class SelectiveStateSpace(_StateMatrixMixer):
         kernels.causal_conv(c, xbc, w["conv"], w["conv_bias"], cache.state, self.matrix_floats, ctx.cu_q, ctx.state_slot,
                             ctx.n_seqs, self._max_q(ctx), act="silu")
         y = torch.empty((n, I), dtype=torch.float32, device=p.device)
-        kernels.gated_scan(y, c[:, I + GN:], c[:, I:I + GN], c[:, :I], dt, None, w["dt_bias"], w["a_log"], w["skip"],
-                           cache.state, ctx.cu_q, ctx.state_slot, ctx.n_seqs, H, self.groups, self.state_size, self.head_dim,
-                           delta=False, k_times_dt=True)
+        self.scan(ctx, c[:, I + GN:], c[:, I:I + GN], c[:, :I], dt, cache.state, y)
         kernels.grouped_gated_norm(out, y, z, w["norm"], I // self.norm_groups, self.eps, gate_act="silu", gate_first=True)
 
     def forward(self, ctx: StepContext, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
