@@ -19,7 +19,7 @@ from .fivedra_bench import fivedra_config
 
 def dizepel_config(width, heads, kv_heads, dim, ssm_heads, vdim, state, groups, ff, vocab, layers=4):
     pair = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
-            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": 4, "softcap": 30.0,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5 / 8, "conv": 4, "softcap": 30.0,
                                "rot": {"dims": dim // 2, "base": 5.0e5, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
                       "right": {"heads": ssm_heads, "vdim": vdim, "state": state, "groups": groups, "conv": 4, "norm_groups": groups}}}
     return {"architecture": "Dizepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.5}, "canon": {"taps": 4},
@@ -88,7 +88,7 @@ def kernels_alone(pk, width=4096, heads=32, kv_heads=8, dim=128, sh=64, sdv=64, 
     r64, a64, b64, h64 = rnd(B, width, dtype=f32), rnd(B, width), rnd(B, width), torch.empty(B, width, dtype=bf, device=dev)
     n64 = dict(norms, h=h64)
     rec(f"stream_layer (pair, norms, filter of {taps} taps) 64 single tokens x {width}",
-        tm.run(lambda: kernels.stream_layer(r64, y=a64, pair=(b64, w, w, 1e-5, 0.5), filt=(filt, fst, slotd), **n64), 3, 10),
+        tm.run(lambda: kernels.stream_layer(r64, y=a64, pair=(b64, w, w, 1e-5, 0.5), filt=(filt.t().contiguous(), fst, slotd), **n64), 3, 10),
         bytes_=B * width * (14 + 8 * (taps - 1)), like="stream_norm of 64 rows below")
     rec(f"stream_norm (Vufolorn) 64 single tokens x {width}",
         tm.run(lambda: kernels.stream_norm(r64, y=a64, w_post=w, layer_scale=w, eps_post=1e-5, h=h64, w_next=w, eps_next=1e-5), 3, 10), bytes_=B * width * 12)

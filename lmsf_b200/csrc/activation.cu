@@ -239,6 +239,8 @@ __global__ void __launch_bounds__(512) poly_norm4_kernel(T* __restrict__ out, co
   const T* row = in + (size_t)blockIdx.x * in_stride;
   T* o = out + (size_t)blockIdx.x * d;
   float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  pdl_launch_dependents();
+  pdl_wait();
   for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
     float z[4];
     ld4(row + i, z);
@@ -279,12 +281,10 @@ LMSF_API int lmsf_poly_norm(void* out, const void* in, int n, int d, long long i
   cudaStream_t s = (cudaStream_t)stream;
   const int threads = d >= 4096 ? 512 : 256;
   if (dtype == LMSF_F32 && rows_take4<float>(in, d, in_stride) && (uintptr_t)out % 16 == 0) {
-    poly_norm4_kernel<float><<<n, threads, 0, s>>>((float*)out, (const float*)in, d, in_stride, coef, eps);
-    return LMSF_LAUNCH_STATUS();
+    return launch_pdl(poly_norm4_kernel<float>, dim3(n), dim3(threads), 0, s, (float*)out, (const float*)in, d, in_stride, coef, eps);
   }
   if (dtype == LMSF_BF16 && rows_take4<bf16>(in, d, in_stride) && (uintptr_t)out % 8 == 0) {
-    poly_norm4_kernel<bf16><<<n, threads, 0, s>>>((bf16*)out, (const bf16*)in, d, in_stride, coef, eps);
-    return LMSF_LAUNCH_STATUS();
+    return launch_pdl(poly_norm4_kernel<bf16>, dim3(n), dim3(threads), 0, s, (bf16*)out, (const bf16*)in, d, in_stride, coef, eps);
   }
   if (dtype == LMSF_F32) poly_norm_kernel<float><<<n, 256, 0, s>>>((float*)out, (const float*)in, d, in_stride, coef, eps);
   else if (dtype == LMSF_BF16) poly_norm_kernel<bf16><<<n, 256, 0, s>>>((bf16*)out, (const bf16*)in, d, in_stride, coef, eps);

@@ -73,15 +73,31 @@ struct ScoreExtras {
   int dist_n;               // dist_n - 1 on) is added to the scaled score
   float softcap;            // > 0: a scaled score s becomes softcap * tanh(s / softcap) before anything else is done to it
 };
-// tanh(x) / x as a polynomial in u = x^2, the series of tanh at 0 through x^9: within 1e-8 of the quotient for |x| <= kTanhSmall
-constexpr float kTanhSmall = 0.25f;
+// tanh(x) / x as a polynomial in u = x^2, of two reaches:
+//   |x| <= kTanhNear: the series of tanh at 0 through x^9, within 1e-8 of the quotient
+//   |x| <= kTanhFar:  the polynomial of degree 9 in u that meets the quotient at the ten Chebyshev points of [0, kTanhFar^2],
+//                     within 2e-8 of it (2e-7 with float32's own rounding)
+// and beyond that 1 - 2 / (1 + e^(2x)) on the special-function unit.
+constexpr float kTanhNear = 0.25f, kTanhFar = 1.5f;
 constexpr float kTanh3 = -1.0f / 3.0f, kTanh5 = 2.0f / 15.0f, kTanh7 = -17.0f / 315.0f, kTanh9 = 62.0f / 2835.0f;
-// tanh(x): the series near 0 (exact relative to x), else 1 - 2 / (1 + e^(2x)) on the special-function unit
-__device__ __forceinline__ float tanh_large(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x * 2.8853900817779268f)); }
+constexpr int kTanhTerms = 10;
+__host__ __device__ constexpr float tanh_far_coef(int i) {
+  constexpr float c[kTanhTerms] = {0.99999998147f, -0.33333167893f, 0.13330850832f, -0.053820780479f, 0.021412750936f,
+                                   -0.0080194525170f, 0.0025848281494f, -6.3165987782e-4f, 9.8872513344e-5f, -7.2078166865e-6f};
+  return c[i];
+}
+constexpr float kTwoLog2e = 2.8853900817779268f;
 __device__ __forceinline__ float tanh_score(float x) {
   const float u = x * x;
-  float t = x * fmaf(u, fmaf(u, fmaf(u, fmaf(u, kTanh9, kTanh7), kTanh5), kTanh3), 1.0f);
-  if (fabsf(x) > kTanhSmall) t = tanh_large(x);
+  float p = tanh_far_coef(kTanhTerms - 1);
+#pragma unroll
+  for (int i = kTanhTerms - 2; i >= 0; --i) p = fmaf(u, p, tanh_far_coef(i));
+  float t = x * p;
+  if (fabsf(x) > kTanhFar) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * kTwoLog2e));
+    t = 1.0f - __fdividef(2.0f, 1.0f + e);
+  }
   return t;
 }
 // The key tiles that a block walks when the window's keys [lo, hi) are joined by the kept first keys [0, keep): tiles

@@ -616,8 +616,8 @@ __global__ void __launch_bounds__(kThreadsTotal, 1) prefill_tc_kernel(const Args
         tmem_wait_ld();
         if constexpr (kCap) {
           // softcap * tanh(s * scale / softcap) in the raw scores' units is s * (tanh(x) / x) with x = s * scale / softcap: the
-          // quotient is a polynomial in x^2 where every score of the warp's rows is small (the usual case: no special function),
-          // else tanh itself is computed
+          // quotient is a polynomial in x^2, a short one where every score of the warp's rows is small and a longer one where all
+          // are within 1.5 caps (no special function in either); else tanh itself is computed, two reciprocals at a time
           const float k = a.scale / a.x.softcap, k2 = k * k;
           float big0 = fmax3(fabsf(sc[0]), fabsf(sc[1]), fabsf(sc[2])), big1 = fmaxf(fabsf(sc[3]), fabsf(sc[4]));
           big1 = fmaxf(big1, fabsf(sc[BN - 1]));
@@ -627,12 +627,30 @@ __global__ void __launch_bounds__(kThreadsTotal, 1) prefill_tc_kernel(const Args
             big1 = fmax3(big1, fabsf(sc[i + 2]), fabsf(sc[i + 3]));
           }
           big0 = fmax3(big0, fabsf(sc[BN - 3]), fabsf(sc[BN - 2]));
-          if (__any_sync(0xffffffffu, fmaxf(big0, big1) * fabsf(k) > kTanhSmall)) {
-            const float inv_k = a.x.softcap / a.scale;
+          const float big = fmaxf(big0, big1) * k;
+          const uint64_t kk = pk2(k2, k2);
+          if (__any_sync(0xffffffffu, !(big <= kTanhFar))) {
+            // tanh(x) = 1 - 2 / (1 + e^(2x)); beyond e^(2x) = 2^60 it is 1 in float32, and two such sums still multiply
+            const float c = k * kTwoLog2e, inv_k = a.x.softcap / a.scale;
 #pragma unroll
-            for (int i = 0; i < BN; ++i) sc[i] = tanh_score(sc[i] * k) * inv_k;
+            for (int i = 0; i < BN; i += 2) {
+              const float d0 = 1.0f + ex2_approx(fminf(sc[i] * c, 60.f)), d1 = 1.0f + ex2_approx(fminf(sc[i + 1] * c, 60.f));
+              const float r = rcp_approx(d0 * d1) * (-2.0f * inv_k);
+              sc[i] = fmaf(r, d1, inv_k);
+              sc[i + 1] = fmaf(r, d0, inv_k);
+            }
+          } else if (__any_sync(0xffffffffu, big > kTanhNear)) {
+#pragma unroll
+            for (int i = 0; i < BN; i += 2) {
+              const uint64_t s2 = pk2(sc[i], sc[i + 1]);
+              const uint64_t u = mul2(mul2(s2, s2), kk);
+              uint64_t p = pk2(tanh_far_coef(kTanhTerms - 1), tanh_far_coef(kTanhTerms - 1));
+#pragma unroll
+              for (int j = kTanhTerms - 2; j >= 0; --j) p = fma2(u, p, pk2(tanh_far_coef(j), tanh_far_coef(j)));
+              upk2(mul2(s2, p), sc[i], sc[i + 1]);
+            }
           } else {
-            const uint64_t kk = pk2(k2, k2), c9 = pk2(kTanh9, kTanh9), c7 = pk2(kTanh7, kTanh7), c5 = pk2(kTanh5, kTanh5),
+            const uint64_t c9 = pk2(kTanh9, kTanh9), c7 = pk2(kTanh7, kTanh7), c5 = pk2(kTanh5, kTanh5),
                            c3 = pk2(kTanh3, kTanh3), one = pk2(1.f, 1.f);
 #pragma unroll
             for (int i = 0; i < BN; i += 2) {

@@ -18,7 +18,10 @@ LMSF_DEFINE_LAST_ERROR(lmsf_conv_rope)
 namespace lmsf {
 
 constexpr int kThreads = 128;
-constexpr int kChunk = 16;          // tokens per block
+#ifndef LMSF_ROPE_CHUNK
+#define LMSF_ROPE_CHUNK 16
+#endif
+constexpr int kChunk = LMSF_ROPE_CHUNK;   // tokens per block
 constexpr int kMaxTaps = 32;
 
 struct ConvRopeArgs {

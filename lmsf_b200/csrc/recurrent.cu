@@ -48,6 +48,8 @@ __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, co
                                    const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                                    long long slot_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slot,
                                    int C, int taps, int act) {
+  pdl_launch_dependents();
+  pdl_wait();
   const int c = blockIdx.x * kConvChannels + threadIdx.x;
   const int s = blockIdx.y;
   const int t0 = cu_q[s], n = cu_q[s + 1] - t0;
@@ -89,7 +91,10 @@ __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, co
 // The same with VEC channels per thread (one 16-byte access of the activation type) and a window that slides in
 // registers: a thread owns its channels for a chunk of kConvVecChunk tokens, reads every input once (and taps - 1 rows
 // before the chunk), and, in a request's first chunk, is also the only reader and writer of its channels' state.
-constexpr int kConvVecChunk = 32;
+#ifndef LMSF_CONV_CHUNK
+#define LMSF_CONV_CHUNK 32
+#endif
+constexpr int kConvVecChunk = LMSF_CONV_CHUNK;
 constexpr int kConvVecThreads = 128;
 
 template <typename T, int VEC> __device__ __forceinline__ void conv_load(const T* p, float (&v)[VEC]);
@@ -122,18 +127,27 @@ __global__ void __launch_bounds__(kConvVecThreads) causal_conv_vec_kernel(
     const int* __restrict__ state_slot, int C, int act) {
   const int c = (blockIdx.x * kConvVecThreads + threadIdx.x) * VEC;
   const int s = blockIdx.y;
-  const int t0 = cu_q[s], n = cu_q[s + 1] - t0;
-  const int lo = blockIdx.z * kConvVecChunk;
-  if (lo >= n || c >= C) return;
-  const int hi = min(n, lo + kConvVecChunk);
-  float* st = state + (size_t)state_slot[s] * slot_stride;      // [TAPS - 1][C]
+  pdl_launch_dependents();
+  if (c >= C) return;
   float wr[TAPS][VEC], b[VEC], win[TAPS > 1 ? TAPS - 1 : 1][VEC];
+  float wl[VEC * TAPS];                          // the channels' weights lie together: 16-byte reads
+#pragma unroll
+  for (int i = 0; i < VEC * TAPS; i += 4) {
+    const float4 x4 = *reinterpret_cast<const float4*>(w + (size_t)c * TAPS + i);
+    wl[i] = x4.x; wl[i + 1] = x4.y; wl[i + 2] = x4.z; wl[i + 3] = x4.w;
+  }
 #pragma unroll
   for (int e = 0; e < VEC; ++e) {
     b[e] = bias ? bias[c + e] : 0.f;
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) wr[j][e] = w[(size_t)(c + e) * TAPS + j];
+    for (int j = 0; j < TAPS; ++j) wr[j][e] = wl[e * TAPS + j];
   }
+  pdl_wait();                                    // what stands above reads weights only, which no kernel of a step writes
+  const int t0 = cu_q[s], n = cu_q[s + 1] - t0;
+  const int lo = blockIdx.z * kConvVecChunk;
+  if (lo >= n) return;
+  const int hi = min(n, lo + kConvVecChunk);
+  float* st = state + (size_t)state_slot[s] * slot_stride;      // [TAPS - 1][C]
   // the TAPS - 1 inputs before the chunk, oldest first: from the portion, or (before its first token) from the state
 #pragma unroll
   for (int j = 0; j < TAPS - 1; ++j) {
@@ -189,10 +203,9 @@ static int launch_conv_vec(void* out, long long out_stride, const void* x, long 
                            float* state, long long slot_stride, const int* cu_q, const int* state_slot, int n_seqs, int max_q, int C,
                            int taps, int act, cudaStream_t s) {
   dim3 grid(ceil_div(C, VEC * kConvVecThreads), n_seqs, ceil_div(max_q, kConvVecChunk));
-#define LMSF_CASE(TP) case TP: causal_conv_vec_kernel<T, VEC, TP><<<grid, kConvVecThreads, 0, s>>>((T*)out, out_stride, (const T*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, act); break;
+#define LMSF_CASE(TP) case TP: return launch_pdl(causal_conv_vec_kernel<T, VEC, TP>, grid, dim3(kConvVecThreads), 0, s, (T*)out, out_stride, (const T*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, act);
   switch (taps) { LMSF_CASE(1) LMSF_CASE(2) LMSF_CASE(3) LMSF_CASE(4) LMSF_CASE(5) LMSF_CASE(6) LMSF_CASE(7) LMSF_CASE(8) default: return LMSF_EBADARG; }
 #undef LMSF_CASE
-  return LMSF_LAUNCH_STATUS();
 }
 
 // ---------------------------------------------------------------------------------------------- scan
@@ -417,6 +430,8 @@ __global__ void __launch_bounds__(BLOCK ? 256 : 128) grouped_gated_norm_reg_kern
   __shared__ float scratch[33];
   const int team = BLOCK ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int me = BLOCK ? threadIdx.x : (threadIdx.x & 31), step = BLOCK ? 256 : 32;
+  pdl_launch_dependents();
+  pdl_wait();
   if (team >= n * n_groups) return;
   const int t = team / n_groups, grp = team % n_groups;
   const float* xr = x + (size_t)t * x_stride + (size_t)grp * gsize;
@@ -481,18 +496,17 @@ LMSF_API int lmsf_causal_conv(void* out, long long out_stride, const void* x, lo
   // 16-byte accesses where the rows allow them (the state's rows are then 16-byte aligned too)
   const int vec = dtype == LMSF_F32 ? 4 : 8;
   if ((dtype == LMSF_F32 || dtype == LMSF_BF16) && taps <= 8 && C % vec == 0 && out_stride % vec == 0 && x_stride % vec == 0 &&
-      ((uintptr_t)out | (uintptr_t)x) % 16 == 0) {
+      ((uintptr_t)out | (uintptr_t)x | (uintptr_t)w) % 16 == 0) {
     if (dtype == LMSF_F32) return launch_conv_vec<float, 4>(out, out_stride, x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, n_seqs, max_q, C, taps, act, s);
     return launch_conv_vec<bf16, 8>(out, out_stride, x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, n_seqs, max_q, C, taps, act, s);
   }
   dim3 grid(ceil_div(C, kConvChannels), n_seqs, ceil_div(max_q, kConvChunk));
   dim3 block(kConvChannels, max_q >= 4 ? 4 : (max_q >= 2 ? 2 : 1));
-#define LMSF_GO(T, M) causal_conv_kernel<T, M><<<grid, block, 0, s>>>((T*)out, out_stride, (const T*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, taps, act)
+#define LMSF_GO(T, M) return launch_pdl(causal_conv_kernel<T, M>, grid, block, 0, s, (T*)out, out_stride, (const T*)x, x_stride, w, bias, state, slot_stride, cu_q, state_slot, C, taps, act)
   if (dtype == LMSF_F32) { if (taps <= 8) LMSF_GO(float, 8); else LMSF_GO(float, kMaxTaps); }
   else if (dtype == LMSF_BF16) { if (taps <= 8) LMSF_GO(bf16, 8); else LMSF_GO(bf16, kMaxTaps); }
-  else LMSF_REFUSE("causal_conv: unknown dtype code %d", dtype);
+  LMSF_REFUSE("causal_conv: unknown dtype code %d", dtype);
 #undef LMSF_GO
-  return LMSF_LAUNCH_STATUS();
 }
 
 // Floats of the scratch that lmsf_gated_scan needs for n_tokens tokens (q and k in the scan's layout, and four floats per
@@ -542,9 +556,9 @@ LMSF_API int lmsf_grouped_gated_norm(void* out, long long out_stride, const floa
   const bool wide = gsize % 4 == 0 && wlen % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && (!gate || gate_stride % 4 == 0) &&
                     ((uintptr_t)x | (uintptr_t)w) % 16 == 0 && ((uintptr_t)out | (uintptr_t)gate) % (4 * esz) == 0;
   const int per = ceil_div(gsize, (block ? 256 : 32) * (wide ? 4 : 1));
-#define LMSF_REG(T, B, P, V) grouped_gated_norm_reg_kernel<T, B, P, V><<<blocks, B ? 256 : 128, 0, s>>>((T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first, out_scale)
-#define LMSF_CASE(T, B, P) if (per <= P) { if (wide) LMSF_REG(T, B, P, 4); else LMSF_REG(T, B, P, 1); return LMSF_LAUNCH_STATUS(); }
-#define LMSF_NARROW(T, B, P) if (!wide && per <= P) { LMSF_REG(T, B, P, 1); return LMSF_LAUNCH_STATUS(); }
+#define LMSF_REG(T, B, P, V) return launch_pdl(grouped_gated_norm_reg_kernel<T, B, P, V>, dim3(blocks), dim3(B ? 256 : 128), 0, s, (T*)out, out_stride, x, x_stride, (const T*)gate, gate_stride, w, wlen, n, n_groups, gsize, eps, gate_silu, gate_first, out_scale)
+#define LMSF_CASE(T, B, P) if (per <= P) { if (wide) LMSF_REG(T, B, P, 4); else LMSF_REG(T, B, P, 1); }
+#define LMSF_NARROW(T, B, P) if (!wide && per <= P) LMSF_REG(T, B, P, 1);
 #define LMSF_PICK(T)                                                                          \
   if (!block) { LMSF_CASE(T, false, 1) LMSF_CASE(T, false, 2) LMSF_CASE(T, false, 4) LMSF_CASE(T, false, 8)  \
                 LMSF_NARROW(T, false, 16) LMSF_NARROW(T, false, 32) }                          \

@@ -1024,9 +1024,9 @@ def stream_layer(res: torch.Tensor, y: Optional[torch.Tensor] = None, pair=None,
                  h: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0,
                  next_centred: bool = False, filt=None):
     """What lies between two branches, for norms that may take the mean off: res += N_post(b); res += vec; h = N_next(res), and
-    behind it, for rows that are single tokens, a short filter over time, h + sum_j f[:, j] * h of the tokens before and its own.
+    behind it, for rows that are single tokens, a short filter over time, h + sum_j f[j] * h of the tokens before and its own.
     N(x) = (x - mean) / sqrt(variance + eps) * w where centred, else x / rms(x) * w.  b = y, or with `pair` (y2, p1, p2, eps,
-    factor) b = factor * (y / rms(y) * p1 + y2 / rms(y2) * p2).  `filt` (f float32 [hidden, taps], state float32 [slots,
+    factor) b = factor * (y / rms(y) * p1 + y2 / rms(y2) * p2).  `filt` (f float32 [taps, hidden], state float32 [slots,
     (taps - 1) * hidden], state_slot int32 [n]): row i is the token of slot state_slot[i], whose inputs are rolled on.
     res: float32 [n, hidden]; y, y2, h: contiguous [n, hidden] of one activation type; vectors float32 [hidden]."""
     n, hidden = res.shape
@@ -1040,10 +1040,10 @@ def stream_layer(res: torch.Tensor, y: Optional[torch.Tensor] = None, pair=None,
     f, taps, state, slots = None, 0, None, None
     if filt is not None:
         f, state, slots = filt
-        taps = f.shape[1]
-        if f.dtype != torch.float32 or f.shape[0] != hidden or not f.is_contiguous() or state.dtype != torch.float32 or \
+        taps = f.shape[0]
+        if f.dtype != torch.float32 or f.shape[1] != hidden or not f.is_contiguous() or state.dtype != torch.float32 or \
                 not state.is_contiguous() or state.dim() != 2 or state.shape[1] < (taps - 1) * hidden or slots.numel() != n:
-            raise KernelError("stream_layer: the filter is float32 [hidden, taps], its state float32 [slots, (taps - 1) * hidden], one slot a row")
+            raise KernelError("stream_layer: the filter is float32 [taps, hidden], its state float32 [slots, (taps - 1) * hidden], one slot a row")
     fn = _func("layer_norm.cu", "lmsf_stream_layer",
                [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_float, c_int, c_void_p, c_void_p,
                 c_void_p, c_float, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p])

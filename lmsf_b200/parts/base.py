@@ -305,7 +305,7 @@ class Shift(Part):
     steps: `state_spec()` says what a slot holds, `forward(ctx, h, state) -> h'` reads and updates it."""
 
     def single_token_filter(self) -> Optional[torch.Tensor]:
-        """float32 [width, taps] when the part is h + sum_j f[:, j] * (rows of the tokens before and the token's own, oldest
+        """float32 [taps, width] when the part is h + sum_j f[j] * (rows of the tokens before and the token's own, oldest
         first) with the rows before, float32 [taps - 1, width], as its state: a step of single tokens may then have it done by the
         kernel that norms the rows.  None otherwise."""
         return None

@@ -20,12 +20,24 @@ norms and the sum into the stream.  A state slot holds the right mixer's state a
 """
 from __future__ import annotations
 
+import os
 from typing import Dict, Optional
 
 import torch
 
 from .base import BranchPair, KVCacheSpec, LayerCache, Mixer, StateSpec, StepContext, WeightSpec, register_part
 from .linear import matmul_tn
+
+
+CONCURRENT = os.environ.get("LMSF_CONCURRENT_MIXERS", "1") != "0"    # steps of single tokens: the two halves on two streams
+_SIDE_STREAMS: Dict[int, "torch.cuda.Stream"] = {}
+
+
+def _side_stream(device) -> "torch.cuda.Stream":
+    index = device.index if device.index is not None else torch.cuda.current_device()
+    if index not in _SIDE_STREAMS:
+        _SIDE_STREAMS[index] = torch.cuda.Stream(device)
+    return _SIDE_STREAMS[index]
 
 
 @register_part("mixer", "parallel_mixers")
@@ -142,6 +154,21 @@ class NormedParallelMixers(Mixer):
         p = matmul_tn(h, self._in, bias=self._in_bias)
         a = torch.empty((ctx.n_tokens, L.q_size), dtype=p.dtype, device=p.device)
         b = torch.empty((ctx.n_tokens, R.inner), dtype=p.dtype, device=p.device)
+        # The halves share nothing but what they read.  A step of single tokens leaves most of the device idle in each of their
+        # kernels, so the right one runs on a stream of its own (in a captured step: a branch of the graph); prompt portions fill
+        # the device and stay on one stream.
+        here = torch.cuda.current_stream(p.device) if CONCURRENT and ctx.decode_only else None
+        side = _side_stream(p.device) if here is not None else None
+        if side is None:
+            R.mix_projected(ctx, p[:, n:n + R.in_size], cache, b)
+            y = matmul_tn(b, R.o)
+        else:
+            side.wait_stream(here)
+            with torch.cuda.stream(side):
+                R.mix_projected(ctx, p[:, n:n + R.in_size], cache, b)
+                y = matmul_tn(b, R.o)
         L.attend_filtered(ctx, p[:, :n], cache, a, self.left_at)
-        R.mix_projected(ctx, p[:, n:n + R.in_size], cache, b)
-        return BranchPair(matmul_tn(a, L.o), matmul_tn(b, R.o), self._w_left, self._w_right, self.eps, self.factor)
+        x = matmul_tn(a, L.o)
+        if side is not None:
+            here.wait_stream(side)      # before anything that either stream made is read, or given back, by the other
+        return BranchPair(x, y, self._w_left, self._w_right, self.eps, self.factor)

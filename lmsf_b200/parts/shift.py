@@ -57,6 +57,7 @@ class FilterShift(Shift):
             raise ValueError(f"a filter of {taps} taps is beyond the kernel (1 to {kernels.CONV_MAX_TAPS})")
         self.filter: Optional[torch.Tensor] = None
         self._f32: Optional[torch.Tensor] = None
+        self._by_tap: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         return {"filter": WeightSpec([(self.hidden_size, self.taps)], keep_fp32=True)}
@@ -66,12 +67,13 @@ class FilterShift(Shift):
 
     def prepare(self, dtype, device) -> None:
         self._f32 = self.filter.float().contiguous()
+        self._by_tap = self._f32.t().contiguous()
 
     def activation_width(self) -> int:
         return self.hidden_size
 
     def single_token_filter(self) -> Optional[torch.Tensor]:
-        return self._f32
+        return self._by_tap
 
     def forward(self, ctx: StepContext, h: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
         out = torch.empty_like(h)

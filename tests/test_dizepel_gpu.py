@@ -81,7 +81,7 @@ def test_one_kernel_joins_norms_adds_norms_again_and_filters(D, dtype):
         if taps:
             f, st = rnd(D, taps), rnd(n + 4, max(1, taps - 1) * D).to(tdt).float()
             state = dev(st.clone())
-            filt = (dev(f), state, i32(slots.tolist()))
+            filt = (dev(f.t().contiguous()), state, i32(slots.tolist()))
         kernels.stream_layer(r, y=dev(y1) if branch else None, pair=(dev(y2), dev(p1), dev(p2), 1e-4, 0.7) if branch == "pair" else None,
                              w_post=dev(wp), eps_post=EPS, post_centred=bool(cp), vec=dev(vec) if use_vec else None, h=h,
                              w_next=dev(wn) if h is not None else None, eps_next=EPS, next_centred=bool(cn), filt=filt)
