@@ -163,7 +163,7 @@ def kernels_alone(pk, width=4096, heads=32, kv_heads=8, dim=128, sh=64, sdv=64, 
     chunks = [(0, c, min(c + n_c, T), j) for j, c in enumerate(range(0, T, n_c))]
     items, spans = ints(chunks), ints([(0, 0, len(chunks), 0)])
     ends = (dtb, a_log, skip, sst)
-    rec(f"scan_chunks (four launches), a prompt of 2048 tokens, {sh} heads of {state} x {sdv}",
+    rec(f"scan_chunks (three launches), a prompt of 2048 tokens, {sh} heads of {state} x {sdv}",
         tm.run(lambda: kernels.scan_chunks(yo, qq, kk, vv, dtr, *ends, cu, slot, 1, sh, groups, state, sdv, items=items, spans=spans), 3, 10),
         fma=5.0 * T * cells, like="gated_scan and matrix_memory below")
     rec(f"gated_scan (Redarax: one chain of tokens), a prompt of 2048 tokens, {sh} heads of {state} x {sdv}",

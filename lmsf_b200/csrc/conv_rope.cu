@@ -19,7 +19,7 @@ namespace lmsf {
 
 constexpr int kThreads = 128;
 #ifndef LMSF_ROPE_CHUNK
-#define LMSF_ROPE_CHUNK 16
+#define LMSF_ROPE_CHUNK 8
 #endif
 constexpr int kChunk = LMSF_ROPE_CHUNK;   // tokens per block
 constexpr int kMaxTaps = 32;
@@ -90,34 +90,46 @@ template <int V> __device__ __forceinline__ void st_vals(bf16* p, const float* v
   }
 }
 
-// TAPS 0: any number of taps, inputs read again for every token.
+// V consecutive values in the stored type, moved in one access
+template <typename T, int V> struct alignas(sizeof(T) * V) Piece { T v[V]; };
+constexpr int kAhead = 4;
+
+// TAPS 0: any number of taps, inputs read again for every token, one block for a whole portion (a chunk may be shorter than the
+// filter, so only the block that rolls the state on may read it).
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(kThreads) conv_rope_kernel(const ConvRopeArgs a) {
   extern __shared__ float cs[];                // [token of the chunk][cos: half | sin: half]
   __shared__ long long row_off[kChunk];        // the token's row inside the cache, kv head 0; negative: no page
   pdl_launch_dependents();
   pdl_wait();
-  const int seq = blockIdx.z, lo = blockIdx.y * kChunk;
+  const int seq = blockIdx.z;
+  int lo = blockIdx.y * kChunk;
   const int t0 = a.cu_q[seq], n = a.cu_q[seq + 1] - t0;
   if (lo >= n) return;
-  const int cnt = min(kChunk, n - lo), half = a.inv_freq ? a.rot_dim / 2 : 0;
-  for (int i = threadIdx.x; i < cnt * half; i += kThreads) {
-    const int t = i / half, p = i % half;
-    float s, c;
-    sincosf((float)a.positions[t0 + lo + t] * a.inv_freq[p], &s, &c);
-    cs[t * 2 * half + p] = c * a.mult;
-    cs[t * 2 * half + half + p] = s * a.mult;
-  }
-  if (threadIdx.x < cnt) {
-    const int pos = a.positions[t0 + lo + threadIdx.x];
-    const int page = a.block_table[(size_t)seq * a.max_blocks + pos / a.block_size];
-    if (page < 0 && blockIdx.x == 0 && a.error_flag) atomicExch(a.error_flag, 2);
-    row_off[threadIdx.x] = page < 0 ? -1 : (long long)page * a.page_stride + (long long)(pos % a.block_size) * a.hd;
-  }
-  __syncthreads();
-  const int per_head = a.hd / (2 * V), item = blockIdx.x * kThreads + threadIdx.x;
-  const int heads = a.n_q_heads + a.n_kv_heads;
-  if (item >= per_head * heads) return;
+  int cnt = min(kChunk, n - lo);
+  const int half = a.inv_freq ? a.rot_dim / 2 : 0;
+  auto stage = [&]() {                         // angles and pages of the chunk's tokens, by the whole block
+    for (int i = threadIdx.x; i < cnt * half; i += kThreads) {
+      const int t = i / half, p = i % half;
+      float s, c;
+      sincosf((float)a.positions[t0 + lo + t] * a.inv_freq[p], &s, &c);
+      cs[t * 2 * half + p] = c * a.mult;
+      cs[t * 2 * half + half + p] = s * a.mult;
+    }
+    if (threadIdx.x < cnt) {
+      const int pos = a.positions[t0 + lo + threadIdx.x];
+      const int page = a.block_table[(size_t)seq * a.max_blocks + pos / a.block_size];
+      if (page < 0 && blockIdx.x == 0 && a.error_flag) atomicExch(a.error_flag, 2);
+      row_off[threadIdx.x] = page < 0 ? -1 : (long long)page * a.page_stride + (long long)(pos % a.block_size) * a.hd;
+    }
+    __syncthreads();
+  };
+  stage();
+  const int per_head = a.hd / (2 * V), heads = a.n_q_heads + a.n_kv_heads;
+  int item = blockIdx.x * kThreads + threadIdx.x;
+  const bool live = item < per_head * heads;
+  if (TAPS > 0 && !live) return;
+  if (!live) item = 0;                         // (TAPS 0: keeps the block's barriers)
   const int head = item / per_head, w = item % per_head;
   const bool turned = w * V < half;            // the first half / V items of a head
   const int tail = a.hd - 2 * half;
@@ -180,21 +192,35 @@ __global__ void __launch_bounds__(kThreads) conv_rope_kernel(const ConvRopeArgs 
     }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) input(lo - (TAPS - 1) + j, win[j]);
-#pragma unroll 2
-    for (int t = lo; t < lo + cnt; ++t) {
-      float cur[2 * V], y[2 * V];
-      input(t, cur);
+    // four tokens' inputs are asked for together, in the stored type
+    for (int tb = lo; tb < lo + cnt; tb += kAhead) {
+      Piece<T, V> in[kAhead][2];
 #pragma unroll
-      for (int e = 0; e < 2 * V; ++e) {
-        float s = 0.f;
-#pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) s = fmaf(wr[j][e], win[j][e], s);
-        y[e] = fmaf(wr[TAPS - 1][e], cur[e], s);
-#pragma unroll
-        for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
-        if (TAPS > 1) win[TAPS > 1 ? TAPS - 2 : 0][e] = cur[e];
+      for (int u = 0; u < kAhead; ++u) {
+        if (tb + u < lo + cnt) {
+          const T* p = x + (size_t)(tb + u) * a.x_stride;
+          in[u][0] = *reinterpret_cast<const Piece<T, V>*>(p + c0);
+          in[u][1] = *reinterpret_cast<const Piece<T, V>*>(p + c1);
+        }
       }
-      emit(t, y);
+#pragma unroll
+      for (int u = 0; u < kAhead; ++u) {
+        if (tb + u >= lo + cnt) break;
+        float cur[2 * V], y[2 * V];
+        ld_vals<V>(in[u][0].v, cur);
+        ld_vals<V>(in[u][1].v, cur + V);
+#pragma unroll
+        for (int e = 0; e < 2 * V; ++e) {
+          float s = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) s = fmaf(wr[j][e], win[j][e], s);
+          y[e] = fmaf(wr[TAPS - 1][e], cur[e], s);
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
+          if (TAPS > 1) win[TAPS > 1 ? TAPS - 2 : 0][e] = cur[e];
+        }
+        emit(tb + u, y);
+      }
     }
     if (lo != 0 || TAPS == 1) return;
 #pragma unroll
@@ -209,20 +235,27 @@ __global__ void __launch_bounds__(kThreads) conv_rope_kernel(const ConvRopeArgs 
       st_vals<V>(st + (size_t)j * C + c1, v + V);
     }
   } else {
-    for (int t = lo; t < lo + cnt; ++t) {
-      float y[2 * V], v[2 * V], wj[2 * V];
+    while (true) {
+      for (int t = lo; live && t < lo + cnt; ++t) {
+        float y[2 * V], v[2 * V], wj[2 * V];
 #pragma unroll
-      for (int e = 0; e < 2 * V; ++e) y[e] = 0.f;
-      for (int j = 0; j < taps; ++j) {
-        input(t - (taps - 1) + j, v);
-        ld_vals<V>(a.w + (size_t)j * C + c0, wj);
-        ld_vals<V>(a.w + (size_t)j * C + c1, wj + V);
+        for (int e = 0; e < 2 * V; ++e) y[e] = 0.f;
+        for (int j = 0; j < taps; ++j) {
+          input(t - (taps - 1) + j, v);
+          ld_vals<V>(a.w + (size_t)j * C + c0, wj);
+          ld_vals<V>(a.w + (size_t)j * C + c1, wj + V);
 #pragma unroll
-        for (int e = 0; e < 2 * V; ++e) y[e] = fmaf(wj[e], v[e], y[e]);
+          for (int e = 0; e < 2 * V; ++e) y[e] = fmaf(wj[e], v[e], y[e]);
+        }
+        emit(t, y);
       }
-      emit(t, y);
+      lo += kChunk;
+      if (lo >= n) break;
+      cnt = min(kChunk, n - lo);
+      __syncthreads();                         // the chunk before has been read
+      stage();
     }
-    if (lo != 0) return;
+    if (!live) return;
     for (int j = 0; j < taps - 1; ++j) {                   // row j takes input n - (taps - 1) + j: a later row, or the portion
       float v[2 * V];
       input(n - (taps - 1) + j, v);
@@ -239,6 +272,7 @@ static int launch_conv_rope(const ConvRopeArgs& a, int n_seqs, int max_q, cudaSt
 #define LMSF_CASE(N) case N: return launch_pdl(conv_rope_kernel<T, V, N>, grid, dim3(kThreads), smem, s, a)
   switch (a.taps) { LMSF_CASE(1); LMSF_CASE(2); LMSF_CASE(3); LMSF_CASE(4); default: break; }
 #undef LMSF_CASE
+  grid.y = 1;
   return launch_pdl(conv_rope_kernel<T, V, 0>, grid, dim3(kThreads), smem, s, a);
 }
 

@@ -35,8 +35,10 @@ constexpr int kConvChannels = 64;    // channels per block (threadIdx.x)
 constexpr int kConvChunk = 256;      // tokens per block along gridDim.z
 constexpr int kMaxTaps = 32;
 enum { kConvPlain = 0, kConvSilu = 1, kConvAddInput = 2 };
-__device__ __forceinline__ float conv_end(float acc, float x, int act) {
-  return act == kConvSilu ? silu_f(acc) : (act == kConvAddInput ? x + acc : acc);
+// (a result that is rounded to bfloat16 next takes the special-function unit's exponential and quotient)
+template <typename T> __device__ __forceinline__ float conv_end(float acc, float x, int act) {
+  if (act == kConvSilu) return sizeof(T) == 2 ? __fdividef(acc, 1.0f + __expf(-acc)) : silu_f(acc);
+  return act == kConvAddInput ? x + acc : acc;
 }
 
 // MAXT: taps that a build holds in registers.
@@ -73,7 +75,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, co
           last = v;                                             // the last tap's input is the token's own
         }
       }
-      out[(size_t)(t0 + t) * out_stride + c] = from_f32<T>(conv_end(acc, last, act));
+      out[(size_t)(t0 + t) * out_stride + c] = from_f32<T>(conv_end<T>(acc, last, act));
     }
   }
   if (blockIdx.z != 0) return;
@@ -92,7 +94,7 @@ __global__ void causal_conv_kernel(T* __restrict__ out, long long out_stride, co
 // registers: a thread owns its channels for a chunk of kConvVecChunk tokens, reads every input once (and taps - 1 rows
 // before the chunk), and, in a request's first chunk, is also the only reader and writer of its channels' state.
 #ifndef LMSF_CONV_CHUNK
-#define LMSF_CONV_CHUNK 32
+#define LMSF_CONV_CHUNK 16
 #endif
 constexpr int kConvVecChunk = LMSF_CONV_CHUNK;
 constexpr int kConvVecThreads = 128;
@@ -168,7 +170,7 @@ __global__ void __launch_bounds__(kConvVecThreads) causal_conv_vec_kernel(
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) a = fmaf(wr[j][e], win[j][e], a);
       a = fmaf(wr[TAPS - 1][e], cur[e], a);
-      acc[e] = conv_end(a, cur[e], act);
+      acc[e] = conv_end<T>(a, cur[e], act);
     }
     conv_store<T, VEC>(out + (size_t)(t0 + t) * out_stride + c, acc);
 #pragma unroll

@@ -1286,8 +1286,8 @@ def scan_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
                 spans: Optional[torch.Tensor] = None):
     """The plain rule of `gated_scan` with k_times_dt on the same state.  items, spans None: every request brings one token, one
     launch.  Else items (int32 [chunks, 4]: request, first token, end token, chunk number) cut long portions into chunks of at most
-    `scan_chunk_tokens()` tokens and spans (int32 [portions, 4]: request, first item, end item, 0) name each portion's chunks; four
-    launches over a scratch that this function allocates."""
+    `scan_chunk_tokens()` tokens and spans (int32 [portions, 4]: request, first item, end item, 0) name each portion's chunks; three
+    (bfloat16) or four launches over a scratch that this function allocates."""
     _rows(q, qk_heads * dk, "scan_chunks: q")
     _rows(k, qk_heads * dk, "scan_chunks: k", q.dtype)
     _rows(v, heads * dv, "scan_chunks: v", q.dtype)
@@ -1313,7 +1313,7 @@ def scan_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
            _i32(spans, "spans"), n_spans, _ptr(scratch), dtype_code(q.dtype), _stream())
     _check(rc, "scan_chunks.cu", "lmsf_scan_chunks")
     if n_chunks:
-        add_launches(3)
+        add_launches(3 if q.dtype == torch.float32 else 2)
 
 
 def grouped_gated_norm(out: torch.Tensor, x: torch.Tensor, gate: Optional[torch.Tensor], w: torch.Tensor, group_size: int,

@@ -205,6 +205,7 @@ MIXERS = [
     (left(6, 2, 144, 0.08, 3, 20.0, rotation(16, 900.0)), right(8, 12, 24, 4, 3, 8), 16),
     (left(5, 5, 64, 0.3, 11, 2.0, rotation(64, 50.0, (2.0, 16, 4.0, 1.0))), right(1, 1, 1, 1, 2, 1), 16),
     (left(1, 1, 2, 0.7, 3, 1.0, rotation(2, 9.0)), right(2, 130, 200, 2, 4, 4), 16),
+    (left(3, 1, 32, 0.3, 32, 4.0, rotation(16, 60.0)), right(3, 9, 40, 3, 20, 1), 16),
 ]
 
 
