@@ -163,6 +163,27 @@ def test_head_weights_are_padded_with_their_filters():
 
 # ----------------------------------------------------------------------------- identities
 
+def test_the_polynomial_of_the_hyperbolic_tangent_in_the_kernels_header_meets_it():
+    """The ten coefficients in attention_mma.cuh are the interpolation of tanh(x) / x in u = x^2 at the Chebyshev points of [0, 1.5^2];
+    evaluated in float32 they give the quotient within float32's rounding."""
+    import os
+    import re
+    import numpy as np
+    from lmsf_b200.csrc import build
+    text = open(os.path.join(build.CSRC_DIR, "attention_mma.cuh")).read()
+    body = re.search(r"c\[kTanhTerms\] = \{([^}]*)\}", text).group(1)
+    coef = [float(x.strip().rstrip("f")) for x in body.replace("\n", " ").split(",")]
+    assert len(coef) == 10 and float(re.search(r"kTanhFar = ([0-9.]+)f", text).group(1)) == 1.5
+    f = lambda u: np.tanh(np.sqrt(u)) / np.sqrt(u)
+    want = np.polynomial.Chebyshev.interpolate(f, 9, domain=[0, 2.25]).convert(kind=np.polynomial.Polynomial).coef
+    assert np.allclose(coef, want, rtol=1e-7, atol=1e-12)
+    u = np.linspace(1e-9, 2.25, 50001).astype(np.float32)
+    p = np.full_like(u, np.float32(coef[-1]))
+    for c in coef[-2::-1]:
+        p = (p.astype(np.float64) * u + np.float32(c)).astype(np.float32)
+    assert float(np.abs(p / f(u.astype(np.float64)) - 1).max()) < 2.5e-7
+
+
 def test_the_series_of_the_hyperbolic_tangent_is_close_where_it_is_used():
     """x (1 + u (-1/3 + u (2/15 + u (-17/315 + u 62/2835)))), u = x^2: within 1e-8 of tanh relative to it up to 1/4."""
     x = torch.linspace(1e-4, 0.25, 5001).double()
